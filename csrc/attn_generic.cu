@@ -5,6 +5,8 @@
 //    the rest pass through), then optional weight-free unit-RMS scaling of q and k per head, append of k / v to the
 //    cache [B][G][T][D] / [B][G][T][Dv].  Token (b, s) goes to slot *cache_len + s at position slot - pad_left[b].
 //    A layer that reads another layer's keys and values runs it for the queries only.
+//  * attn_prep_all_kernel — the same for designs that norm q (and k) over all heads together and mix the values with another
+//    layer's; two CTAs per token.
 //  * attn_rows_kernel   — 16 queries of one head per CTA against key / value tiles of 32 rows staged in shared memory
 //    (one key per lane for the scores, one value column per lane for the output), online softmax in fp32, causal over
 //    slots [pad_left[b], slot], optional per-head output gate sigmoid(g).  Prompts of any length; exact path for
@@ -215,6 +217,114 @@ __global__ void __launch_bounds__(128) rotary_slice_kernel(const T* __restrict__
   }
 }
 
+// Preparation of designs whose q / k norm runs over ALL channels of the projection (weights [H*D] / [G*D]) before the rotation,
+// and whose values may be mixed with another layer's values of the same token: v <- (1 - l) v + l v_first.  Two CTAs per
+// token: the queries; the keys and values.  Sums of squares first, then the rows again (L1 hits) with the rotation and the stores.
+struct PrepAllParams {
+  const float* y; int ldy;
+  int q_off, k_off, v_off;
+  int S, H, G, D, Dv, T;
+  int rot, layout;
+  const float* cos_t; const float* sin_t; int max_pos;
+  float eps;
+  const int* cache_len; const int* pad_left;
+  const float* bias;                // fp32, indexed like the columns of y, or nullptr
+  const float* v_first; int ldvf;   // fp32 [M][G*Dv] (row pitch ldvf), or nullptr
+  int vec;                          // 16-byte accesses are aligned: D, Dv, rot, ldy and the offsets are multiples of four
+};
+
+constexpr int PA_THREADS = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(PA_THREADS) attn_prep_all_kernel(PrepAllParams p, const T* __restrict__ qw, const T* __restrict__ kw,
+                                                                   const T* __restrict__ v_lambda, T* __restrict__ q_out,
+                                                                   T* __restrict__ kc, T* __restrict__ vc) {
+  pdl_wait();                      // programmatic dependent launch: nothing is read before the predecessor is done
+  pdl_launch_dependents();
+  __shared__ float red[33];
+  const int m = blockIdx.x, b = m / p.S, s = m % p.S;
+  const bool is_q = blockIdx.y == 0;
+  const int slot = (p.cache_len ? *p.cache_len : 0) + s;
+  int pos = slot - (p.pad_left ? p.pad_left[b] : 0);
+  pos = pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos);
+  const float* yr = p.y + (size_t)m * p.ldy;
+  const int n = (is_q ? p.H : p.G) * p.D, off = is_q ? p.q_off : p.k_off;
+  const float* src = yr + off;
+  const float* bs = p.bias ? p.bias + off : nullptr;
+  const T* w = is_q ? qw : kw;
+  const float* ct = p.cos_t + (size_t)pos * (p.rot / 2);
+  const float* st = p.sin_t + (size_t)pos * (p.rot / 2);
+  // channel c of the row -> where it goes
+  auto dst_of = [&](int c) -> T* {
+    return is_q ? q_out + (size_t)m * n + c : kc + (((size_t)b * p.G + c / p.D) * p.T + slot) * p.D + c % p.D;
+  };
+  float ss = 0.0f;
+  if (p.vec) {
+    for (int c = 4 * threadIdx.x; c < n; c += 4 * PA_THREADS) {
+      float v[4];
+      load4(src + c, v);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { if (bs) v[e] += bs[c + e]; ss += v[e] * v[e]; }
+    }
+  } else {
+    for (int c = threadIdx.x; c < n; c += PA_THREADS) { const float v = src[c] + (bs ? bs[c] : 0.0f); ss += v * v; }
+  }
+  const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)n + p.eps);
+  if (p.vec && (p.layout == 0 || p.rot == 0)) {
+    for (int c = 4 * threadIdx.x; c < n; c += 4 * PA_THREADS) {
+      float v[4], wv[4];
+      load4(src + c, v);
+      load4(w + c, wv);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { if (bs) v[e] += bs[c + e]; v[e] = v[e] * r * wv[e]; }
+      const int d = c % p.D;
+      if (d < p.rot) {                                     // two whole pairs: rot is a multiple of four here
+        const float2 cs = *reinterpret_cast<const float2*>(ct + d / 2), sn = *reinterpret_cast<const float2*>(st + d / 2);
+        const float o[4] = {v[0] * cs.x - v[1] * sn.x, v[1] * cs.x + v[0] * sn.x, v[2] * cs.y - v[3] * sn.y, v[3] * cs.y + v[2] * sn.y};
+        store4(dst_of(c), o);
+      } else {
+        store4(dst_of(c), v);
+      }
+    }
+  } else {
+    auto val = [&](int c) { return (src[c] + (bs ? bs[c] : 0.0f)) * r * to_f(w[c]); };
+    for (int c = threadIdx.x; c < n; c += PA_THREADS) {
+      const int d = c % p.D;
+      float o;
+      if (d >= p.rot) o = val(c);
+      else if (p.layout == 0) o = (d & 1) ? val(c) * ct[d >> 1] + val(c - 1) * st[d >> 1] : val(c) * ct[d >> 1] - val(c + 1) * st[d >> 1];
+      else {
+        const int half = p.rot / 2;
+        o = d < half ? val(c) * ct[d] - val(c + half) * st[d] : val(c) * ct[d - half] + val(c - half) * st[d - half];
+      }
+      *dst_of(c) = from_f<T>(o);
+    }
+  }
+  if (is_q) return;
+  const float lam = p.v_first ? to_f(*v_lambda) : 0.0f;
+  const float* vs = yr + p.v_off;
+  const float* vb = p.bias ? p.bias + p.v_off : nullptr;
+  const float* vf = p.v_first ? p.v_first + (size_t)m * p.ldvf : nullptr;
+  const int nv = p.G * p.Dv;
+  auto vdst = [&](int c) { return vc + (((size_t)b * p.G + c / p.Dv) * p.T + slot) * p.Dv + c % p.Dv; };
+  if (p.vec) {
+    for (int c = 4 * threadIdx.x; c < nv; c += 4 * PA_THREADS) {
+      float v[4], f[4];
+      load4(vs + c, v);
+      if (vf) load4(vf + c, f);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { if (vb) v[e] += vb[c + e]; if (vf) v[e] = (1.0f - lam) * v[e] + lam * f[e]; }
+      store4(vdst(c), v);
+    }
+  } else {
+    for (int c = threadIdx.x; c < nv; c += PA_THREADS) {
+      float v = vs[c] + (vb ? vb[c] : 0.0f);
+      if (vf) v = (1.0f - lam) * v + lam * vf[c];
+      *vdst(c) = from_f<T>(v);
+    }
+  }
+}
+
 struct AttnParams {
   int B, S, H, G, D, Dv, T;
   int ldk, ldv;                     // row pitch of the key / value cache in elements (>= D / Dv: the two may be columns of one row)
@@ -231,7 +341,13 @@ struct AttnParams {
   const float* sink_logit;          // [H] fp32: the extra term of the denominator is exp(sink_logit[h]) instead of exp(0) (with sink = 1)
   const float* vcos; const float* vsin; int v_max_pos, v_layout;   // [v_max_pos][Dv/2]: the cached values were rotated at their own
                                     // positions; every head's sum is rotated back by the query's position (pairs as v_layout)
+  float softcap;                    // > 0: scores become softcap * tanh(score / softcap)
 };
+
+__device__ __forceinline__ float attn_score(float dot, float scale, float softcap) {
+  const float s = dot * scale;
+  return softcap > 0.0f ? softcap * tanhf(s / softcap) : s;
+}
 
 // first slot a query at slot hi_q of a row whose sequence starts at slot lo may see
 __device__ __forceinline__ int attn_first_visible(const AttnParams& p, int lo, int hi_q) {
@@ -277,7 +393,7 @@ constexpr int AT_MAXV = 16;         // value columns per lane: Dv <= 512
 // scores of one block of 32 keys (lane = key), then the block's contribution to the output (lane = value column)
 template <typename T>
 __device__ __forceinline__ void attn_block(const float* __restrict__ qs, const T* __restrict__ kbase, const T* __restrict__ vbase,
-                                           int j0, int lo, int hi, int D, int Dv, int ldk, int ldv, float scale, float& mrun,
+                                           int j0, int lo, int hi, int D, int Dv, int ldk, int ldv, float scale, float softcap, float& mrun,
                                            float& lrun, float (&acc)[AT_MAXV]) {
   const int lane = threadIdx.x & 31;
   const int j = j0 + lane;
@@ -286,7 +402,7 @@ __device__ __forceinline__ void attn_block(const float* __restrict__ qs, const T
     const T* kr = kbase + (size_t)j * ldk;
     float d = 0.0f;
     for (int c = 0; c < D; ++c) d = fmaf(qs[c], to_f(kr[c]), d);
-    sc = d * scale;
+    sc = attn_score(d, scale, softcap);
   }
   const float mnew = fmaxf(mrun, warp_max(sc));
   if (mnew == -INFINITY) return;                       // nothing visible in this block (uniform across the warp)
@@ -424,7 +540,7 @@ __global__ void __launch_bounds__(AR_WARPS * 32) attn_rows_kernel(AttnParams p, 
     for (int qi = 0; qi < AR_QW; ++qi) {
       pj[qi] = 0.0f;
       if (!on[qi]) continue;
-      const float sc = (j >= lo_q[qi] && j <= hi_q[qi]) ? (d0[qi] + d1[qi]) * p.scale : -INFINITY;
+      const float sc = (j >= lo_q[qi] && j <= hi_q[qi]) ? attn_score(d0[qi] + d1[qi], p.scale, p.softcap) : -INFINITY;
       const float mnew = fmaxf(mrun[qi], warp_max(sc));
       if (mnew == -INFINITY) continue;
       const float corr = mrun[qi] == -INFINITY ? 0.0f : expf(mrun[qi] - mnew);
@@ -503,7 +619,7 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_kernel(AttnParams p
   const T* vbase = vc + (size_t)b * p.v_bs + (size_t)g * p.v_hs;
   float mrun = -INFINITY, lrun = 0.0f, acc[AT_MAXV] = {};
   for (int j0 = (lo & ~31) + 32 * warp; j0 <= hi; j0 += 32 * AD_WARPS)
-    attn_block<T>(qs, kbase, vbase, j0, lo, hi, p.D, p.Dv, p.ldk, p.ldv, p.scale, mrun, lrun, acc);
+    attn_block<T>(qs, kbase, vbase, j0, lo, hi, p.D, p.Dv, p.ldk, p.ldv, p.scale, p.softcap, mrun, lrun, acc);
   if (lane == 0) { ml[2 * warp] = mrun; ml[2 * warp + 1] = lrun; }
 #pragma unroll
   for (int i = 0; i < AT_MAXV; ++i) {
@@ -606,7 +722,7 @@ __global__ void __launch_bounds__(AS_WARPS * 32) attn_split_kernel(AttnParams p,
     for (int qi = 0; qi < AS_RW; ++qi) {
       pj[qi] = 0.0f;
       if (warp + AS_WARPS * qi >= R) continue;           // warp-uniform
-      const float sc = vis ? (d0[qi] + d1[qi]) * p.scale : -INFINITY;
+      const float sc = vis ? attn_score(d0[qi] + d1[qi], p.scale, p.softcap) : -INFINITY;
       const float mnew = fmaxf(mrun[qi], warp_max(sc));
       if (mnew == -INFINITY) continue;
       const float corr = mrun[qi] == -INFINITY ? 0.0f : expf(mrun[qi] - mnew);
@@ -752,6 +868,28 @@ extern "C" JL_API int jl_attn_prep_ex(const float* y, int ldy, int q_off, int k_
   return attn_prep_launch(p, q_out, k_cache, v_cache, dtype, stream);
 }
 
+extern "C" JL_API int jl_attn_prep_all(const float* y, int ldy, int q_off, int k_off, int v_off, void* q_out, void* k_cache,
+                                       void* v_cache, const float* cos_t, const float* sin_t, int max_pos, int rot, int layout,
+                                       const void* q_norm_w, const void* k_norm_w, float eps, const int* cache_len,
+                                       const int* pad_left, int B, int S, int H, int G, int D, int Dv, int T_cap, const float* bias,
+                                       const float* v_first, int ldvf, const void* v_lambda, int dtype, void* stream) {
+  JL_CHECK_ARG(B >= 1 && S >= 1 && H >= 1 && G >= 1 && H % G == 0 && D >= 1 && Dv >= 1, "jl_attn_prep_all: bad shape");
+  JL_CHECK_ARG(rot >= 0 && rot <= D && rot % 2 == 0 && (layout == 0 || layout == 1), "jl_attn_prep_all: rot=%d of D=%d, layout %d", rot,
+               D, layout);
+  JL_CHECK_ARG(q_norm_w != nullptr && k_norm_w != nullptr && max_pos >= 1, "jl_attn_prep_all: both norm weights are needed");
+  JL_CHECK_ARG(v_first == nullptr || (v_lambda != nullptr && ldvf >= G * Dv), "jl_attn_prep_all: mixed values need the weight and a pitch");
+  const int vec = D % 4 == 0 && Dv % 4 == 0 && rot % 4 == 0 && ldy % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 && v_off % 4 == 0 &&
+                  (v_first == nullptr || ldvf % 4 == 0) &&
+                  ((uintptr_t)y | (uintptr_t)v_first | (uintptr_t)q_norm_w | (uintptr_t)k_norm_w | (uintptr_t)q_out | (uintptr_t)k_cache |
+                   (uintptr_t)v_cache) % 16 == 0;
+  PrepAllParams p{y, ldy, q_off, k_off, v_off, S, H, G, D, Dv, T_cap, rot, layout, cos_t, sin_t, max_pos, eps, cache_len, pad_left, bias,
+                  v_first, ldvf, vec};
+  JL_DISPATCH_DTYPE(dtype, JL_LAUNCH_PDL(attn_prep_all_kernel<T>, dim3(B * S, 2), dim3(PA_THREADS), 0, (cudaStream_t)stream, p,
+                                         (const T*)q_norm_w, (const T*)k_norm_w, (const T*)v_lambda, (T*)q_out, (T*)k_cache, (T*)v_cache));
+  JL_CUDA(cudaGetLastError());
+  return JL_OK;
+}
+
 extern "C" JL_API int jl_attn_generic_splits(int B, int H, int G, int T_cap) {
   if (G <= 0) return 0;
   const int nblk = (H / G + AS_WARPS * AS_RW - 1) / (AS_WARPS * AS_RW);      // blocks of query heads per key/value head
@@ -767,17 +905,18 @@ static int attn_launch(const void* q, const void* k_cache, const void* v_cache, 
                        int ldv, int window, float scale, float* scratch, int splits, int dtype, void* stream,
                        long long k_bs = 0, long long k_hs = 0, long long v_bs = 0, long long v_hs = 0, int sink = 0,
                        float* out32 = nullptr, int chunk = 0, const float* sink_logit = nullptr, const float* vcos = nullptr,
-                       const float* vsin = nullptr, int v_max_pos = 0, int v_layout = 0) {
+                       const float* vsin = nullptr, int v_max_pos = 0, int v_layout = 0, float softcap = 0.0f) {
   JL_CHECK_ARG(B >= 1 && S >= 1 && G >= 1 && H % G == 0, "jl_attn_generic: H=%d not a multiple of G=%d", H, G);
   JL_CHECK_ARG(Dv <= 32 * AT_MAXV, "jl_attn_generic: value size %d above %d", Dv, 32 * AT_MAXV);
   JL_CHECK_ARG(ldk >= D && ldv >= Dv && window >= 0, "jl_attn_generic: bad pitch %d / %d or window %d", ldk, ldv, window);
   if (k_bs == 0 && k_hs == 0) { k_hs = (long long)T_cap * ldk; k_bs = k_hs * G; }
   if (v_bs == 0 && v_hs == 0) { v_hs = (long long)T_cap * ldv; v_bs = v_hs * G; }
+  JL_CHECK_ARG(softcap >= 0.0f, "jl_attn_generic: softcap %f", softcap);
   JL_CHECK_ARG(chunk >= 0 && (sink_logit == nullptr || sink), "jl_attn_generic: chunk %d, a sink logit without a sink", chunk);
   JL_CHECK_ARG(vcos == nullptr || (vsin != nullptr && Dv % 2 == 0 && v_max_pos >= 1 && (v_layout == 0 || v_layout == 1)),
                "jl_attn_generic: rotated values need both tables and an even Dv=%d", Dv);
   AttnParams p{B, S, H, G, D, Dv, T_cap, ldk, ldv, k_bs, k_hs, v_bs, v_hs, window, scale, cache_len, pad_left, gate, ldg, sink, out32,
-               chunk, sink_logit, vcos, vsin, v_max_pos, v_layout};
+               chunk, sink_logit, vcos, vsin, v_max_pos, v_layout, softcap};
   cudaStream_t st = (cudaStream_t)stream;
   if (S == 1 && scratch != nullptr && splits >= 1 && splits <= 64) {
     const int dp = ((D + 3) & ~3) + 4;
@@ -836,17 +975,17 @@ extern "C" JL_API int jl_attn_windowed(const void* q, const void* k_cache, const
 }
 
 // Everything the attention kernels take: gate (fp32 pre-activation, column h of row m, pitch ldg), window, blocks of `chunk`
-// positions, a sink (score 0, or sink_logit[h]), values cached rotated (v_cos / v_sin [v_max_pos][Dv/2], pairs as v_layout).
+// positions, capped scores (softcap > 0), a sink (score 0, or sink_logit[h]), values cached rotated (v_cos / v_sin [v_max_pos][Dv/2], pairs as v_layout).
 extern "C" JL_API int jl_attn_masked(const void* q, const void* k_cache, const void* v_cache, void* out, const float* gate, int ldg,
                                      const int* cache_len, const int* pad_left, int B, int S, int H, int G, int D, int Dv, int T_cap,
                                      int ldk, int ldv, long long k_bs, long long k_hs, long long v_bs, long long v_hs, int window,
-                                     int chunk, float scale, float* scratch, int splits, int sink, const float* sink_logit,
+                                     int chunk, float scale, float softcap, float* scratch, int splits, int sink, const float* sink_logit,
                                      const float* v_cos, const float* v_sin, int v_max_pos, int v_layout, float* out32, int dtype,
                                      void* stream) {
   JL_CHECK_ARG(out != nullptr || out32 != nullptr, "jl_attn_masked: no output");
   return attn_launch(q, k_cache, v_cache, out, gate, ldg, cache_len, pad_left, B, S, H, G, D, Dv, T_cap, ldk, ldv, window, scale,
                      scratch, splits, dtype, stream, k_bs, k_hs, v_bs, v_hs, sink, out32, chunk, sink_logit, v_cos, v_sin, v_max_pos,
-                     v_layout);
+                     v_layout, softcap);
 }
 
 extern "C" JL_API int jl_latent_prep(const float* y, int ldy, int q_off, int q_rank, int kv_off, int kv_rank, int rot_dim, int rot,

@@ -41,6 +41,9 @@ struct FlashParams {
   const float* gate; int ldg;       // fp32 pre-activation of a sigmoid per (token, head) on the output (column h of row m), or nullptr
   const float* vcos; const float* vsin; int v_max_pos;   // [v_max_pos][64]: the cached values were rotated at their own positions over
                                     // all 128 channels (pairs m, m + 64); every row of the output is rotated back by its position
+  int window;                       // > 0: a query sees itself and the window - 1 slots before it
+  float cap_log2, cap_rate;         // cap_log2 > 0: scores are capped, s -> cap tanh(s / cap): cap log2(e) and the factor 2 scale log2(e) / cap
+                                    // that turns a raw product into the exponent of e^(2 s / cap) in base 2
 };
 
 __device__ __forceinline__ void fence_proxy_async() {
@@ -265,8 +268,8 @@ constexpr float F2_RESCALE_THRESHOLD = 8.0f;                 // log2 units
 // P_TMEM: the probabilities go back to the tensor core through TMEM (tcgen05.st over the columns of the
 // score tile they were computed from; A operand of P·V read from TMEM) instead of swizzled shared memory:
 // no generic→async proxy fence, and the softmax warps no longer wait for P·V_{j-1} before producing P_j.
-// MASKED: the kernel also reads the block size, sink, gate and value-rotation fields of its parameters (one more instance, so that
-// plain causal attention keeps its register budget).
+// MASKED: the kernel also reads the block size, window, cap, sink, gate and value-rotation fields of its parameters (one more
+// instance, so that plain causal attention keeps its register budget).
 template <bool P_TMEM, bool MASKED = false>
 __global__ void __launch_bounds__(256, 2)   // 256: caps registers at 128 so that two 6-warp CTAs (allocated as 8) fit
 flash_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
@@ -321,6 +324,7 @@ flash_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
   const int q_hi = min(q0 + FA_BM, p.S) - 1;
   int lo_cta = pad;                                        // first key any query of this tile sees (its first query's)
   if (MASKED && p.chunk > 0 && p.start + q0 >= pad) lo_cta = pad + (p.start + q0 - pad) / p.chunk * p.chunk;
+  if (MASKED && p.window > 0) lo_cta = max(lo_cta, p.start + q0 - p.window + 1);
   const int first_tile = lo_cta / F2_BN;
   const int last_tile = (p.start + q_hi) / F2_BN;
   const int n_tiles = last_tile - first_tile + 1 > 0 ? last_tile - first_tile + 1 : 0;
@@ -405,6 +409,11 @@ flash_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
       if (q_slot >= pad) lo_row = pad + (q_slot - pad) / p.chunk * p.chunk;
       if (q_last >= pad) lo_warp = pad + (q_last - pad) / p.chunk * p.chunk;
     }
+    if (MASKED && p.window > 0) {
+      lo_row = max(lo_row, q_slot - p.window + 1);
+      lo_warp = max(lo_warp, p.start + q0 + quarter * 32 + 31 - p.window + 1);
+    }
+    const float to_log2 = (MASKED && p.cap_log2 > 0.f) ? 1.0f : p.scale_log2;     // capped scores are already in the log2 domain
 
     for (int j = 0; j < n_tiles; ++j) {
       const int key0 = (first_tile + j) * F2_BN;
@@ -415,6 +424,15 @@ flash_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
       tc::tmem_ld32(tS(j) + lane_off, v0);
       tc::tmem_ld32(tS(j) + lane_off + 32, v1);
       tc::tmem_ld_wait();
+      if (MASKED && p.cap_log2 > 0.f) {
+        // cap tanh(s / cap) = cap - 2 cap / (1 + e^(2 s / cap)), absolute error a few 1e-7 of the cap (tanh.approx has 5e-4)
+        const float twice = 2.0f * p.cap_log2;
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          v0[i] = __float_as_uint(p.cap_log2 - __fdividef(twice, 1.0f + exp2f(__uint_as_float(v0[i]) * p.cap_rate)));
+          v1[i] = __float_as_uint(p.cap_log2 - __fdividef(twice, 1.0f + exp2f(__uint_as_float(v1[i]) * p.cap_rate)));
+        }
+      }
       if (need_mask) {
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
@@ -426,7 +444,7 @@ flash_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
 #pragma unroll
       for (int i = 0; i < 32; ++i)
         mx4[i & 3] = fmaxf(mx4[i & 3], fmaxf(__uint_as_float(v0[i]), __uint_as_float(v1[i])));
-      const float t = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2;
+      const float t = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * to_log2;
       // P·V_{j-1} must be complete before the P tile in shared memory is overwritten
       if (!P_TMEM && j > 0) {
         tc::mbar_wait(o_full, (j - 1) & 1);
@@ -460,10 +478,10 @@ flash_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
         uint32_t w[32];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          const float a0 = exp2f(fmaf(__uint_as_float(v0[2 * i]), p.scale_log2, -m_safe));
-          const float a1 = exp2f(fmaf(__uint_as_float(v0[2 * i + 1]), p.scale_log2, -m_safe));
-          const float b0 = exp2f(fmaf(__uint_as_float(v1[2 * i]), p.scale_log2, -m_safe));
-          const float b1 = exp2f(fmaf(__uint_as_float(v1[2 * i + 1]), p.scale_log2, -m_safe));
+          const float a0 = exp2f(fmaf(__uint_as_float(v0[2 * i]), to_log2, -m_safe));
+          const float a1 = exp2f(fmaf(__uint_as_float(v0[2 * i + 1]), to_log2, -m_safe));
+          const float b0 = exp2f(fmaf(__uint_as_float(v1[2 * i]), to_log2, -m_safe));
+          const float b1 = exp2f(fmaf(__uint_as_float(v1[2 * i + 1]), to_log2, -m_safe));
           psum += (a0 + a1) + (b0 + b1);
           w[i] = pack_bf16(a0, a1);
           w[16 + i] = pack_bf16(b0, b1);
@@ -478,7 +496,7 @@ flash_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
           for (int i = 0; i < 16; ++i) {
             const float s0 = __uint_as_float(c == 0 ? v0[2 * i] : v1[2 * i]);
             const float s1 = __uint_as_float(c == 0 ? v0[2 * i + 1] : v1[2 * i + 1]);
-            const float p0 = exp2f(fmaf(s0, p.scale_log2, -m_safe)), p1 = exp2f(fmaf(s1, p.scale_log2, -m_safe));
+            const float p0 = exp2f(fmaf(s0, to_log2, -m_safe)), p1 = exp2f(fmaf(s1, to_log2, -m_safe));
             psum += p0 + p1;
             w[i] = pack_bf16(p0, p1);
           }
@@ -620,39 +638,44 @@ extern "C" JL_API int jl_flash_prefill_occupancy(int smem_override) {
 
 static int flash_launch(const void* q, const void* k_cache, const void* v_cache, const int* pad_left, void* out, int B, int S, int nh,
                         int nkv, int hd, int T, int start, float scale, void* stream, int chunk, int sink, const float* sink_logit,
-                        const float* gate, int ldg, const float* vcos, const float* vsin, int v_max_pos);
+                        const float* gate, int ldg, const float* vcos, const float* vsin, int v_max_pos, int window, float softcap);
 
 extern "C" JL_API int jl_flash_prefill(const void* q, const void* k_cache, const void* v_cache,
                                        const int* cache_len_ptr, const int* pad_left, void* out, int B, int S,
                                        int nh, int nkv, int hd, int T, int start, float scale, void* stream) {
   (void)cache_len_ptr;
   return flash_launch(q, k_cache, v_cache, pad_left, out, B, S, nh, nkv, hd, T, start, scale, stream, 0, 0, nullptr, nullptr, 0, nullptr,
-                      nullptr, 0);
+                      nullptr, 0, 0, 0.0f);
 }
 
-// The tcgen05 kernel (128-wide heads) with blocks of `chunk` positions, a sink in the denominator (logit per head), a sigmoid gate
-// per (token, head) and the turn back of values that were cached rotated at their own positions (pairs m, m + 64).
+// The tcgen05 kernel (128-wide heads) with blocks of `chunk` positions, a window, capped scores, a sink in the denominator (logit per head), a sigmoid gate
+// per (token, head) and the turn back of values that were cached rotated at their own positions (pairs m, m + 64).  64-wide heads
+// run the warp-level tensor-core kernel with the same options (no value rotation).
 extern "C" JL_API int jl_flash_prefill_masked(const void* q, const void* k_cache, const void* v_cache, const int* pad_left, void* out,
                                               int B, int S, int nh, int nkv, int hd, int T, int start, float scale, int chunk,
                                               int sink, const float* sink_logit, const float* gate, int ldg, const float* v_cos,
-                                              const float* v_sin, int v_max_pos, void* stream) {
-  JL_CHECK_ARG(hd == FA_HD, "jl_flash_prefill_masked: head_dim=%d (128 is built)", hd);
+                                              const float* v_sin, int v_max_pos, int window, float softcap, void* stream) {
+  JL_CHECK_ARG(hd == FA_HD || (hd == 64 && v_cos == nullptr), "jl_flash_prefill_masked: head_dim=%d (128, and 64 without rotated values)", hd);
+  JL_CHECK_ARG(window >= 0 && softcap >= 0.0f, "jl_flash_prefill_masked: window %d, softcap %f", window, softcap);
   JL_CHECK_ARG(chunk >= 0 && (sink_logit == nullptr || sink) && (gate == nullptr || ldg >= nh),
                "jl_flash_prefill_masked: chunk %d, sink %d, gate pitch %d", chunk, sink, ldg);
   JL_CHECK_ARG(v_cos == nullptr || (v_sin != nullptr && v_max_pos >= 1), "jl_flash_prefill_masked: rotated values need both tables");
   return flash_launch(q, k_cache, v_cache, pad_left, out, B, S, nh, nkv, hd, T, start, scale, stream, chunk, sink, sink_logit, gate, ldg,
-                      v_cos, v_sin, v_max_pos);
+                      v_cos, v_sin, v_max_pos, window, softcap);
 }
 
 static int flash_launch(const void* q, const void* k_cache, const void* v_cache, const int* pad_left, void* out, int B, int S, int nh,
                         int nkv, int hd, int T, int start, float scale, void* stream, int chunk, int sink, const float* sink_logit,
-                        const float* gate, int ldg, const float* vcos, const float* vsin, int v_max_pos) {
-  const bool extras = chunk > 0 || sink || gate != nullptr || vcos != nullptr;
+                        const float* gate, int ldg, const float* vcos, const float* vsin, int v_max_pos, int window, float softcap) {
+  const bool extras = chunk > 0 || window > 0 || softcap > 0.0f || sink || gate != nullptr || vcos != nullptr;
   // 64-wide heads (1B-class LLaMA-architecture models) go to the warp-level tensor-core kernel (prefill_attn_mma.cu);
   // JLLAMA_PREFILL_MMA=1 sends head_dim 128 there too (A/B against the tcgen05 kernel below)
   static const bool force_mma = [] { const char* e = getenv("JLLAMA_PREFILL_MMA"); return e && e[0] == '1'; }();
   if (!extras && (hd == 64 || (force_mma && hd == 128)))
     return jl_prefill_attn_mma(q, k_cache, v_cache, pad_left, out, B, S, nh, nkv, hd, T, start, scale, stream);
+  if (hd == 64)
+    return jl_prefill_attn_mma_masked(q, k_cache, v_cache, pad_left, out, B, S, nh, nkv, hd, T, start, scale, window, chunk, softcap, sink,
+                                      sink_logit, gate, ldg, stream);
   JL_CHECK_ARG(hd == FA_HD, "jl_flash_prefill: head_dim=%d (64 and 128 are built)", hd);
   JL_CHECK_ARG(nkv > 0 && nh % nkv == 0, "jl_flash_prefill: nh=%d not a multiple of nkv=%d", nh, nkv);
   JL_CHECK_ARG(start >= 0 && start + S <= T, "jl_flash_prefill: start=%d + S=%d exceeds cache capacity %d", start, S, T);
@@ -668,7 +691,8 @@ static int flash_launch(const void* q, const void* k_cache, const void* v_cache,
   rc = make_tmap_3d_bf16(&tv, v_cache, (uint64_t)B * nkv, T, hd, (uint64_t)T * hd, hd, bn);
   if (rc) return rc;
   FlashParams p{(__nv_bfloat16*)out, pad_left, B, S, nh, nkv, T, start, scale * 1.4426950408889634f,
-                chunk, sink, sink_logit, gate, ldg, vcos, vsin, v_max_pos};
+                chunk, sink, sink_logit, gate, ldg, vcos, vsin, v_max_pos, window, softcap * 1.4426950408889634f,
+                softcap > 0.0f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.0f};
   dim3 grid((S + FA_BM - 1) / FA_BM, nh, B);
   if (use_v1) {
     const size_t smem = 6 * FA_TILE_BYTES + 128 + 1024;

@@ -48,10 +48,19 @@ struct GlaParams {
   // aux[m * ld_aux + h] and the value row is scaled by aux[m * ld_aux + H + h]
   int qk_div;                          // heads per q / k head (1: every head has its own)
   const float* aux; int ld_aux;
+  // linear attention over activated projections: q, k and v pass `act` (ACT_NONE: as they are)
+  int act;
+  // matrix memory (jl_mlstm_scan): the last `ones` (0 or 1) of the Dv columns are not in y but constantly one before the value
+  // scale, so the state's last column is the normaliser n and the last read-out column n . q
+  int ones;
 };
 
-__device__ __forceinline__ float scan_value_scale(const GlaParams& p, size_t m, int h) {
-  return p.aux ? p.aux[m * p.ld_aux + p.H + h] : 1.0f;
+__device__ __forceinline__ float scan_value(const GlaParams& p, size_t m, int h, int c) {
+  if (c >= p.Dv) return 0.0f;
+  const int dv = p.Dv - p.ones;
+  float v = c < dv ? p.y[m * p.ldy + p.v_off + h * dv + c] : 1.0f;
+  if (p.act != ACT_NONE) v = apply_act(v, p.act, 0.0f, 0.0f);
+  return p.aux ? v * p.aux[m * p.ld_aux + p.H + h] : v;
 }
 
 // q, k and alpha of channel d of head h for the token whose projection row is yr (position pos).
@@ -68,6 +77,9 @@ __device__ __forceinline__ void scan_channel(const GlaParams& p, size_t m, int h
     const float* st = p.sin_t + (size_t)pos * (p.rot / 2);
     qv = rotary_channel(qh, d, p.rot, p.layout, ct, st) * p.q_scale;
     kv = rotary_channel(kh, d, p.rot, p.layout, ct, st) * p.k_scale;
+  } else if (p.act != ACT_NONE) {
+    qv = apply_act(qh[d], p.act, 0.0f, 0.0f) * p.q_scale;
+    kv = apply_act(kh[d], p.act, 0.0f, 0.0f) * p.k_scale;
   } else {
     qv = qh[d] * p.q_scale;
     kv = kh[d] * p.k_scale;
@@ -105,6 +117,7 @@ __global__ void __launch_bounds__(GS_THREADS, 3) gla_scan_kernel(GlaParams p, co
   float* vs = as + GS_TC * DS;                               // [TC][cols]
   float* zs = vs + GS_TC * cols;                             // [TC][R]
 
+  const bool idle = (int)blockIdx.x * cols + (tid & ~31) / P >= p.Dv;      // warp-uniform: no column of this warp exists
   float st[GS_DP];
   const int d0 = part * GS_DP;
   float* sbase = p.state + (((size_t)b * p.H + h) * p.D) * p.Dv;
@@ -123,8 +136,7 @@ __global__ void __launch_bounds__(GS_THREADS, 3) gla_scan_kernel(GlaParams p, co
     }
     for (int i = tid; i < nt * cols; i += GS_THREADS) {
       const int t = i / cols, c = blockIdx.x * cols + i % cols;
-      const size_t mt = (size_t)(b * p.S + s0 + t);
-      vs[i] = c < p.Dv ? p.y[mt * p.ldy + p.v_off + h * p.Dv + c] * scan_value_scale(p, mt, h) : 0.0f;
+      vs[i] = scan_value(p, (size_t)(b * p.S + s0 + t), h, c);
     }
     __syncthreads();
     for (int i = tid; i < nt * P * GS_DP; i += GS_THREADS) {
@@ -136,6 +148,7 @@ __global__ void __launch_bounds__(GS_THREADS, 3) gla_scan_kernel(GlaParams p, co
       qs[at] = qv; ks[at] = kv; as[at] = av;
     }
     __syncthreads();
+    if (idle) continue;
     for (int t = 0; t < nt; ++t) {
       const float v = vs[t * cols + lcol];
       const float4* qt = reinterpret_cast<const float4*>(qs + t * DS + part * GS_PITCH);
@@ -213,7 +226,7 @@ __global__ void __launch_bounds__(128) gla_prep_kernel(GlaParams p, const T* __r
   const int dvp = (p.Dv + 3) & ~3;
   for (int i = threadIdx.x; i < p.H * dvp; i += blockDim.x) {
     const int h = i / dvp, c = i % dvp;
-    out[(size_t)h * RF + 3 * P * pitch + c] = c < p.Dv ? yr[p.v_off + h * p.Dv + c] * scan_value_scale(p, (size_t)m, h) : 0.0f;
+    out[(size_t)h * RF + 3 * P * pitch + c] = scan_value(p, (size_t)m, h, c);
   }
 }
 
@@ -235,6 +248,7 @@ __global__ void __launch_bounds__(GS_THREADS, 2) gla_stream_kernel(GlaParams p, 
   const int tid = threadIdx.x, part = tid % P, grp = tid / P;
   const int col0 = blockIdx.x * cols + grp * C;                         // first of this thread's C columns
   const int h = blockIdx.y, b = blockIdx.z / p.NC, chunk = blockIdx.z % p.NC;
+  const bool idle = (int)blockIdx.x * cols + (tid & ~31) / P * C >= p.Dv;  // warp-uniform: no column of this warp exists
   const int QKA = 3 * P * PITCH;                                        // floats of q | k | alpha per token
   const int SF = QKA + cols;                                            // floats per token in a stage
   const int RF = gla_record_floats(P, DP, p.Dv);
@@ -274,7 +288,7 @@ __global__ void __launch_bounds__(GS_THREADS, 2) gla_stream_kernel(GlaParams p, 
   for (int s0 = first; s0 < t_end; s0 += GS_TS, stage ^= 1) {
     if (s0 + GS_TS < t_end) { issue(s0 + GS_TS, stage ^ 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
     __syncthreads();
-    const int nt = min(GS_TS, t_end - s0);
+    const int nt = idle ? 0 : min(GS_TS, t_end - s0);
     const float* base = smem + (size_t)stage * GS_TS * SF;
     for (int t = 0; t < nt; ++t) {
       const float* tk = base + t * SF;
@@ -468,5 +482,28 @@ extern "C" JL_API int jl_ssd_scan(const float* u, int ldu, int q_off, int k_off,
   GlaParams p{u, ldu, q_off, k_off, v_off, 0, B, S, H, D, Dv, 0, 1, 1.0f, 1.0f, cache_len, pad_left, state, o};
   p.k_scale = 1.0f;
   p.qk_div = H / G; p.aux = aux; p.ld_aux = 2 * H;
+  return launch_scan(p, nullptr, nullptr, ws, DT_F32, stream);
+}
+
+// One fixed decay per head over projections that pass an activation (no rotation, no scale): S_t = decay_h S_(t-1) + k_t v_t^T.
+extern "C" JL_API int jl_activated_scan(const float* y, int ldy, int q_off, int k_off, int v_off, const float* head_decay, int act,
+                                        float* state, float* o, const int* cache_len, const int* pad_left, int B, int S, int H, int D,
+                                        int Dv, float* ws, void* stream) {
+  JL_CHECK_ARG(B >= 1 && S >= 1 && H >= 1 && D >= 1 && Dv >= 1 && head_decay != nullptr, "jl_activated_scan: bad shape");
+  JL_CHECK_ARG(act == ACT_NONE || act == ACT_SILU || act == ACT_SIGMOID || act == ACT_GELU_TANH || act == ACT_RELU2,
+               "jl_activated_scan: activation %d", act);
+  GlaParams p{y, ldy, q_off, k_off, v_off, 0, B, S, H, D, Dv, 0, 1, 1.0f, 1.0f, cache_len, pad_left, state, o};
+  p.head_decay = head_decay; p.k_scale = 1.0f; p.act = act;
+  return launch_scan(p, nullptr, nullptr, ws, DT_F32, stream);
+}
+
+// Matrix memory: decay and value scale per (token, head) from aux [M][ld_aux] (columns h and H + h), Dv value columns of y followed by
+// one column of ones; state [B][H][D][Dv + 1], o [M][H][Dv + 1] (last column: n . q).  ws as for Dv + 1 columns.
+extern "C" JL_API int jl_mlstm_scan(const float* y, int ldy, int q_off, int k_off, int v_off, const float* aux, int ld_aux, float q_scale,
+                                    float* state, float* o, const int* cache_len, const int* pad_left, int B, int S, int H, int D,
+                                    int Dv, float* ws, void* stream) {
+  JL_CHECK_ARG(B >= 1 && S >= 1 && H >= 1 && D >= 1 && Dv >= 1 && aux != nullptr && ld_aux >= 2 * H, "jl_mlstm_scan: bad shape");
+  GlaParams p{y, ldy, q_off, k_off, v_off, 0, B, S, H, D, Dv + 1, 0, 1, q_scale, 1.0f, cache_len, pad_left, state, o};
+  p.k_scale = 1.0f; p.aux = aux; p.ld_aux = ld_aux; p.ones = 1;
   return launch_scan(p, nullptr, nullptr, ws, DT_F32, stream);
 }

@@ -32,6 +32,12 @@ struct PrefillMmaParams {
   __nv_bfloat16* out;                  // [B, S, nh * HD]
   int S, nh, nkv, T, start;
   float scale_log2;
+  // the MASKED instances (all off when zero / null): window, blocks of `chunk` positions, capped scores (as in flash_prefill.cu),
+  // a sink in the denominator (logit per head, or 0), a sigmoid gate per (token, head)
+  int window, chunk;
+  float cap_log2, cap_rate;
+  int sink; const float* sink_logit;
+  const float* gate; int ldg;
 };
 
 __device__ __forceinline__ void pm_mma(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
@@ -48,7 +54,7 @@ __device__ __forceinline__ uint32_t pm_prmt(uint32_t a, uint32_t b, uint32_t sel
 }
 __device__ __forceinline__ uint32_t pm_w(const uint4& v, int i) { return i == 0 ? v.x : (i == 1 ? v.y : (i == 2 ? v.z : v.w)); }
 
-template <int HD>
+template <int HD, bool MASKED>
 __global__ void __launch_bounds__(PM_WARPS * 32) prefill_attn_mma_kernel(const PrefillMmaParams p) {
   constexpr int CH = HD / 32;                  // 16-byte chunks of a row per thread (Q, K)
   constexpr int KS = HD / 16;                  // k-steps of S = Q Kᵀ
@@ -96,7 +102,20 @@ __global__ void __launch_bounds__(PM_WARPS * 32) prefill_attn_mma_kernel(const P
   const __nv_bfloat16* vbase = p.vc + head_off + 8 * g;
   const int lim0 = p.start + r0, lim1 = p.start + r1;                      // causal limit of each row (inclusive)
 
-  for (int base = first; base <= kmax; base += PM_KEYS) {
+  // first key each row sees; the warp starts at its first row's (bounds grow with the row)
+  int lo0 = first, lo1 = first, begin = first;
+  if (MASKED) {
+    auto bound = [&](int lim) {
+      int lo = first;
+      if (p.window > 0) lo = max(lo, lim - p.window + 1);
+      if (p.chunk > 0 && lim >= first) lo = max(lo, first + (lim - first) / p.chunk * p.chunk);
+      return lo;
+    };
+    lo0 = bound(lim0); lo1 = bound(lim1); begin = bound(p.start + q0);
+  }
+  const float to_log2 = (MASKED && p.cap_log2 > 0.f) ? 1.0f : p.scale_log2;
+
+  for (int base = begin; base <= kmax; base += PM_KEYS) {
     uint4 kr[NT][CH], vr[NB][4][VH];
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
@@ -127,10 +146,15 @@ __global__ void __launch_bounds__(PM_WARPS * 32) prefill_attn_mma_kernel(const P
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
       const int key = base + 8 * j + 2 * t;
-      c[j][0] = key <= lim0 ? c[j][0] * p.scale_log2 : -INFINITY;
-      c[j][1] = key + 1 <= lim0 ? c[j][1] * p.scale_log2 : -INFINITY;
-      c[j][2] = key <= lim1 ? c[j][2] * p.scale_log2 : -INFINITY;
-      c[j][3] = key + 1 <= lim1 ? c[j][3] * p.scale_log2 : -INFINITY;
+      if (MASKED && p.cap_log2 > 0.f) {
+        const float twice = 2.0f * p.cap_log2;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) c[j][i] = p.cap_log2 - __fdividef(twice, 1.0f + exp2f(c[j][i] * p.cap_rate));
+      }
+      c[j][0] = key <= lim0 && (!MASKED || key >= lo0) ? c[j][0] * to_log2 : -INFINITY;
+      c[j][1] = key + 1 <= lim0 && (!MASKED || key + 1 >= lo0) ? c[j][1] * to_log2 : -INFINITY;
+      c[j][2] = key <= lim1 && (!MASKED || key >= lo1) ? c[j][2] * to_log2 : -INFINITY;
+      c[j][3] = key + 1 <= lim1 && (!MASKED || key + 1 >= lo1) ? c[j][3] * to_log2 : -INFINITY;
       mx0 = fmaxf(mx0, fmaxf(c[j][0], c[j][1]));
       mx1 = fmaxf(mx1, fmaxf(c[j][2], c[j][3]));
     }
@@ -175,7 +199,16 @@ __global__ void __launch_bounds__(PM_WARPS * 32) prefill_attn_mma_kernel(const P
   // ---- normalise and store: thread (g, t) holds, per row and 64-column half, d = 64 hh + 16 t + [0, 16)
   l[0] += __shfl_xor_sync(0xffffffffu, l[0], 1); l[0] += __shfl_xor_sync(0xffffffffu, l[0], 2);
   l[1] += __shfl_xor_sync(0xffffffffu, l[1], 1); l[1] += __shfl_xor_sync(0xffffffffu, l[1], 2);
-  const float inv0 = l[0] > 0.f ? 1.f / l[0] : 0.f, inv1 = l[1] > 0.f ? 1.f / l[1] : 0.f;
+  if (MASKED && p.sink) {                          // a row that sees a key has a finite maximum
+    const float z = (p.sink_logit ? p.sink_logit[h] : 0.f) * 1.4426950408889634f;
+    if (l[0] > 0.f) l[0] += exp2f(z - m[0]);
+    if (l[1] > 0.f) l[1] += exp2f(z - m[1]);
+  }
+  float inv0 = l[0] > 0.f ? 1.f / l[0] : 0.f, inv1 = l[1] > 0.f ? 1.f / l[1] : 0.f;
+  if (MASKED && p.gate != nullptr) {
+    if (r0 < p.S) inv0 *= 1.0f / (1.0f + __expf(-p.gate[((size_t)b * p.S + r0) * p.ldg + h]));
+    if (r1 < p.S) inv1 *= 1.0f / (1.0f + __expf(-p.gate[((size_t)b * p.S + r1) * p.ldg + h]));
+  }
 #pragma unroll
   for (int hh = 0; hh < VH; ++hh) {
     uint32_t w0[8], w1[8];                   // columns 16 t + [0, 8) come from c0 of tiles e, + [8, 16) from c1
@@ -203,18 +236,38 @@ __global__ void __launch_bounds__(PM_WARPS * 32) prefill_attn_mma_kernel(const P
 
 using namespace jl;
 
+static int mma_launch(const PrefillMmaParams& p, int B, int hd, bool masked, void* stream) {
+  const int S = p.S, nh = p.nh;
+  JL_CHECK_ARG(hd == 64 || hd == 128, "jl_prefill_attn_mma: head_dim=%d (64 and 128 are built)", hd);
+  JL_CHECK_ARG(p.nkv > 0 && nh % p.nkv == 0, "jl_prefill_attn_mma: nh=%d not a multiple of nkv=%d", nh, p.nkv);
+  JL_CHECK_ARG(p.start >= 0 && p.start + S <= p.T, "jl_prefill_attn_mma: start=%d + S=%d exceeds cache capacity %d", p.start, S, p.T);
+  if (B * S == 0) return JL_OK;
+  const dim3 grid((S + PM_WARPS * PM_ROWS - 1) / (PM_WARPS * PM_ROWS), nh, B);
+  auto s = (cudaStream_t)stream;
+  if (masked) JL_CUDA(launch_pdl(prefill_attn_mma_kernel<64, true>, grid, dim3(PM_WARPS * 32), 0, s, p));
+  else if (hd == 64) JL_CUDA(launch_pdl(prefill_attn_mma_kernel<64, false>, grid, dim3(PM_WARPS * 32), 0, s, p));
+  else JL_CUDA(launch_pdl(prefill_attn_mma_kernel<128, false>, grid, dim3(PM_WARPS * 32), 0, s, p));
+  return JL_OK;
+}
+
 extern "C" JL_API int jl_prefill_attn_mma(const void* q, const void* k_cache, const void* v_cache, const int* pad_left,
                                           void* out, int B, int S, int nh, int nkv, int hd, int T, int start, float scale,
                                           void* stream) {
-  JL_CHECK_ARG(hd == 64 || hd == 128, "jl_prefill_attn_mma: head_dim=%d (64 and 128 are built)", hd);
-  JL_CHECK_ARG(nkv > 0 && nh % nkv == 0, "jl_prefill_attn_mma: nh=%d not a multiple of nkv=%d", nh, nkv);
-  JL_CHECK_ARG(start >= 0 && start + S <= T, "jl_prefill_attn_mma: start=%d + S=%d exceeds cache capacity %d", start, S, T);
-  if (B * S == 0) return JL_OK;
   PrefillMmaParams p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, pad_left,
                      (__nv_bfloat16*)out, S, nh, nkv, T, start, scale * 1.4426950408889634f};
-  const dim3 grid((S + PM_WARPS * PM_ROWS - 1) / (PM_WARPS * PM_ROWS), nh, B);
-  auto s = (cudaStream_t)stream;
-  if (hd == 64) JL_CUDA(launch_pdl(prefill_attn_mma_kernel<64>, grid, dim3(PM_WARPS * 32), 0, s, p));
-  else JL_CUDA(launch_pdl(prefill_attn_mma_kernel<128>, grid, dim3(PM_WARPS * 32), 0, s, p));
-  return JL_OK;
+  return mma_launch(p, B, hd, false, stream);
+}
+
+extern "C" JL_API int jl_prefill_attn_mma_masked(const void* q, const void* k_cache, const void* v_cache, const int* pad_left, void* out,
+                                                 int B, int S, int nh, int nkv, int hd, int T, int start, float scale, int window,
+                                                 int chunk, float softcap, int sink, const float* sink_logit, const float* gate,
+                                                 int ldg, void* stream) {
+  JL_CHECK_ARG(hd == 64, "jl_prefill_attn_mma_masked: head_dim=%d (64 is built)", hd);
+  JL_CHECK_ARG(window >= 0 && chunk >= 0 && softcap >= 0.0f && (sink_logit == nullptr || sink) && (gate == nullptr || ldg >= nh),
+               "jl_prefill_attn_mma_masked: window %d, chunk %d, softcap %f", window, chunk, softcap);
+  PrefillMmaParams p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, pad_left,
+                     (__nv_bfloat16*)out, S, nh, nkv, T, start, scale * 1.4426950408889634f, window, chunk,
+                     softcap * 1.4426950408889634f, softcap > 0.0f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.0f, sink,
+                     sink_logit, gate, ldg};
+  return mma_launch(p, B, hd, true, stream);
 }

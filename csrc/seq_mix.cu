@@ -9,6 +9,9 @@
 //  * glu_act_kernel         — gated activations of a fused gate | up product (act(g) * u; the clamped sigmoid form).
 //  * talk_mix_kernel        — attention weights mixed across heads, applied to the per-(head, value head) weighted sums.
 //  * ssd_gates_kernel       — step size, decay and value scale of a selective state space layer.
+//  * mlstm_gates_kernel, mlstm_finish_kernel — what a matrix memory with exponential gates has around its scan: decay, value
+//    scale and denominator floor from a running maximum (a max-plus scan over time); division by the denominator, per-head
+//    norm, weight and gate.
 //
 // Token (b, s) of a call sits at slot *cache_len + s and position slot - pad_left[b]; negative positions are padding.
 #include <stdint.h>
@@ -62,14 +65,16 @@ __global__ void __launch_bounds__(128) embed_pair_norm_kernel(const int* __restr
   for (int i = threadIdx.x; i < W; i += blockDim.x) orow[i] = orow[i] * rn * to_f(norm_w[i]);     // own elements only
 }
 
-constexpr int CC_MAX_TAPS = 8;
+constexpr int CC_FEW_TAPS = 8, CC_MAX_TAPS = 32;      // two instances: the history of a channel lives in registers
 constexpr int CC_CHUNK = 64;       // tokens per CTA along time
 
 // grid (channel blocks, rows, time chunks); a thread owns one channel and walks its chunk with the last taps-1 inputs in
 // registers.  Only the first chunk reads the state (chunks are at least taps-1 tokens long) and it is also the one that
 // replaces it, from the read-only inputs and the old values it holds in registers.
-template <typename T>
+// in_bias (fp32 per channel) belongs to the projection: it is part of every input, but not of the zeros before the start.
+template <typename T, int MT>
 __global__ void __launch_bounds__(128) causal_conv_kernel(const float* __restrict__ y, int ldy, int col0, int C,
+                                                          const float* __restrict__ in_bias,
                                                           const T* __restrict__ w, const T* __restrict__ bias,
                                                           float* __restrict__ state, float* __restrict__ out, int ldo,
                                                           const int* __restrict__ cache_len, const int* __restrict__ pad_left,
@@ -81,21 +86,22 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const float* __restric
   const int s0 = blockIdx.z * chunk, s1 = min(S, s0 + chunk);
   const int first = (pad_left ? pad_left[b] : 0) - (cache_len ? *cache_len : 0);      // tokens before it are padding
   const int nh = taps - 1;
-  float wv[CC_MAX_TAPS], hist[CC_MAX_TAPS];        // hist[j]: the input j + 1 tokens back
+  float wv[MT], hist[MT];        // hist[j]: the input j + 1 tokens back
 #pragma unroll
-  for (int j = 0; j < CC_MAX_TAPS; ++j) { wv[j] = j < taps ? to_f(w[(size_t)c * taps + j]) : 0.0f; hist[j] = 0.0f; }
+  for (int j = 0; j < MT; ++j) { wv[j] = j < taps ? to_f(w[(size_t)c * taps + j]) : 0.0f; hist[j] = 0.0f; }
   const float bv = bias ? to_f(bias[c]) : 0.0f;
   float* st = state + (size_t)b * nh * C + c;      // st[i * C]: the input taps-1-i tokens before this call's first
-  auto input = [&](int s) { return s >= first ? y[(size_t)(b * S + s) * ldy + col0 + c] : 0.0f; };
+  const float ib = in_bias ? in_bias[c] : 0.0f;
+  auto input = [&](int s) { return s >= first ? y[(size_t)(b * S + s) * ldy + col0 + c] + ib : 0.0f; };
 #pragma unroll
-  for (int j = 0; j < CC_MAX_TAPS; ++j) {
+  for (int j = 0; j < MT; ++j) {
     if (j >= nh) break;
     const int s = s0 - 1 - j;
     hist[j] = s >= 0 ? input(s) : st[(size_t)(nh + s) * C];
   }
   if (blockIdx.z == 0) {                           // s0 == 0: hist holds the whole old state; write the new one
 #pragma unroll
-    for (int i = 0; i < CC_MAX_TAPS; ++i) {
+    for (int i = 0; i < MT; ++i) {
       if (i >= nh) break;
       const int s = S - nh + i;                    // the token this state slot holds after the call
       float v;
@@ -103,7 +109,7 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const float* __restric
       else {                                       // still a token of an earlier call: old slot i + S, i.e. -s - 1 tokens back
         v = 0.0f;
 #pragma unroll
-        for (int j = 0; j < CC_MAX_TAPS; ++j) if (j == -s - 1) v = hist[j];
+        for (int j = 0; j < MT; ++j) if (j == -s - 1) v = hist[j];
       }
       st[(size_t)i * C] = v;
     }
@@ -112,10 +118,10 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const float* __restric
     const float xin = input(s);
     float acc = fmaf(wv[taps - 1], xin, bv);
 #pragma unroll
-    for (int j = 0; j < CC_MAX_TAPS; ++j) if (j < nh) acc = fmaf(wv[nh - 1 - j], hist[j], acc);
+    for (int j = 0; j < MT; ++j) if (j < nh) acc = fmaf(wv[nh - 1 - j], hist[j], acc);
     out[(size_t)(b * S + s) * ldo + c] = s >= first ? apply_act(acc, act, 0.0f, 0.0f) : 0.0f;
 #pragma unroll
-    for (int j = CC_MAX_TAPS - 1; j > 0; --j) hist[j] = hist[j - 1];
+    for (int j = MT - 1; j > 0; --j) hist[j] = hist[j - 1];
     hist[0] = xin;
   }
 }
@@ -255,9 +261,128 @@ __global__ void ssd_gates_kernel(const float* __restrict__ y, int ldy, int dt_of
   aux[(size_t)m * 2 * H + H + h] = dt;
 }
 
+// Gates of a matrix memory, one CTA per (row, head).  With i = cap tanh((y_i + b_i) / cap), f = logsigmoid(cap tanh((y_f + b_f) / cap))
+// the running maximum is m_t = max(f_t + m_(t-1), i_t); a stretch of tokens maps m to max(F + m, I), and two stretches compose to
+// (F1 + F2, max(I1 + F2, I2)): a thread folds MG_TPT consecutive tokens, the CTA scans the threads, then every thread
+// walks its tokens again from its incoming m.  aux [M][3H]: decay exp(f + m_(t-1) - m_t) | value scale exp(i - m_t) | floor exp(-m_t).
+// Padding tokens change nothing and get (1, 0, 1).
+constexpr int MG_THREADS = 256, MG_TPT = 8;
+
+__device__ __forceinline__ float cap_tanh(float z, float cap) { return cap * tanhf(z / cap); }
+
+template <typename T>
+__global__ void __launch_bounds__(MG_THREADS) mlstm_gates_kernel(const float* __restrict__ y, int ldy, int i_off, int f_off,
+                                                                 const T* __restrict__ ib, const T* __restrict__ fb, float cap,
+                                                                 float* __restrict__ m_state, float* __restrict__ aux,
+                                                                 const int* __restrict__ cache_len, const int* __restrict__ pad_left,
+                                                                 int S, int H) {
+  pdl_wait();                      // programmatic dependent launch: nothing is read before the predecessor is done
+  pdl_launch_dependents();
+  __shared__ float wF[MG_THREADS / 32], wI[MG_THREADS / 32];
+  const int h = blockIdx.x, b = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int first = max(0, (pad_left ? pad_left[b] : 0) - (cache_len ? *cache_len : 0));
+  const float bi = to_f(ib[h]), bf = to_f(fb[h]);
+  float m_in = m_state[(size_t)b * H + h];                   // read by every thread; replaced by the last one after the loop's barrier
+  for (int s0 = 0; s0 < S; s0 += MG_THREADS * MG_TPT) {
+    float iv[MG_TPT], fv[MG_TPT];
+    const int sb = s0 + threadIdx.x * MG_TPT;
+    float F = 0.0f, I = -INFINITY;
+#pragma unroll
+    for (int t = 0; t < MG_TPT; ++t) {
+      const int s = sb + t;
+      iv[t] = -INFINITY; fv[t] = 0.0f;
+      if (s >= first && s < S) {
+        const float* yr = y + (size_t)(b * S + s) * ldy;
+        iv[t] = yr[i_off + h];
+        fv[t] = yr[f_off + h];
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < MG_TPT; ++t) {
+      const int s = sb + t;
+      if (s >= first && s < S) {
+        iv[t] = cap_tanh(iv[t] + bi, cap);
+        const float z = cap_tanh(fv[t] + bf, cap);
+        fv[t] = z >= 0.0f ? -log1pf(expf(-z)) : z - log1pf(expf(z));
+      }
+      F += fv[t];
+      I = fmaxf(I + fv[t], iv[t]);
+    }
+    // inclusive scan over the warp, then the warps' totals
+    for (int off = 1; off < 32; off <<= 1) {
+      const float Fp = __shfl_up_sync(0xffffffffu, F, off), Ip = __shfl_up_sync(0xffffffffu, I, off);
+      if (lane >= off) { I = fmaxf(Ip + F, I); F += Fp; }
+    }
+    if (lane == 31) { wF[warp] = F; wI[warp] = I; }
+    __syncthreads();
+    float m = m_in;                                          // the maximum this thread's tokens start from
+    for (int w = 0; w < warp; ++w) m = fmaxf(m + wF[w], wI[w]);
+    float m_next = m_in;                                     // and the one the next stretch starts from
+    for (int w = 0; w < MG_THREADS / 32; ++w) m_next = fmaxf(m_next + wF[w], wI[w]);
+    const float Fe = __shfl_up_sync(0xffffffffu, F, 1), Ie = __shfl_up_sync(0xffffffffu, I, 1);
+    if (lane > 0) m = fmaxf(m + Fe, Ie);
+#pragma unroll
+    for (int t = 0; t < MG_TPT; ++t) {
+      const int s = sb + t;
+      if (s >= S) break;
+      float* a = aux + (size_t)(b * S + s) * 3 * H + h;
+      if (s < first) { a[0] = 1.0f; a[H] = 0.0f; a[2 * H] = 1.0f; continue; }
+      const float mn = fmaxf(fv[t] + m, iv[t]);
+      a[0] = expf(fv[t] + m - mn);
+      a[H] = expf(iv[t] - mn);
+      a[2 * H] = expf(-mn);
+      m = mn;
+    }
+    m_in = m_next;
+    __syncthreads();                                         // the warps' totals are free again
+  }
+  if (threadIdx.x == 0) m_state[(size_t)b * H + h] = m_in;
+}
+
+// One warp per (token, head); o fp32 [M][H][V + 1], the last column is n . q:
+// v = o / (max(|n . q|, floor) + 1e-6);  out = v / sqrt(mean(v^2) + eps) * w[h, :] * act(gate)
+template <typename T>
+__global__ void mlstm_finish_kernel(const float* __restrict__ o, const float* __restrict__ aux, const T* __restrict__ w,
+                                    const float* __restrict__ gate, int ldg, T* __restrict__ out, int M, int H, int V, float eps,
+                                    int gate_act) {
+  pdl_wait();                      // programmatic dependent launch: nothing is read before the predecessor is done
+  pdl_launch_dependents();
+  const int wid = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (wid >= M * H) return;
+  const int m = wid / H, h = wid % H;
+  const float* orow = o + ((size_t)m * H + h) * (V + 1);
+  const float inv = 1.0f / (fmaxf(fabsf(orow[V]), aux[(size_t)m * 3 * H + 2 * H + h]) + 1e-6f);
+  float ss = 0.0f;
+  for (int i = lane; i < V; i += 32) { const float v = orow[i] * inv; ss += v * v; }
+  const float r = inv / sqrtf(warp_sum(ss) / (float)V + eps);
+  const float* grow = gate + (size_t)m * ldg + (size_t)h * V;
+  for (int i = lane; i < V; i += 32)
+    out[((size_t)m * H + h) * V + i] = from_f<T>(orow[i] * r * to_f(w[h * V + i]) * apply_act(grow[i], gate_act, 0.f, 0.f));
+}
+
 }  // namespace jl
 
 using namespace jl;
+
+extern "C" JL_API int jl_mlstm_gates(const float* y, int ldy, int i_off, int f_off, const void* i_bias, const void* f_bias, float cap,
+                                     float* m_state, float* aux, const int* cache_len, const int* pad_left, int B, int S, int H,
+                                     int dtype, void* stream) {
+  JL_CHECK_ARG(B >= 1 && S >= 1 && H >= 1 && cap > 0.0f, "jl_mlstm_gates: bad shape or cap %f", cap);
+  JL_DISPATCH_DTYPE(dtype, JL_LAUNCH_PDL(mlstm_gates_kernel<T>, dim3(H, B), dim3(MG_THREADS), 0, stream, y, ldy, i_off, f_off,
+                                         (const T*)i_bias, (const T*)f_bias, cap, m_state, aux, cache_len, pad_left, S, H));
+  JL_CUDA(cudaGetLastError());
+  return JL_OK;
+}
+
+extern "C" JL_API int jl_mlstm_finish(const float* o, const float* aux, const void* w, const float* gate, int ldg, void* out, int M,
+                                      int H, int V, float eps, int gate_act, int dtype, void* stream) {
+  JL_CHECK_ARG(M >= 1 && H >= 1 && V >= 1 && ldg >= H * V && w != nullptr, "jl_mlstm_finish: bad shape M=%d H=%d V=%d", M, H, V);
+  const int warps = 4, blocks = (M * H + warps - 1) / warps;
+  JL_DISPATCH_DTYPE(dtype, JL_LAUNCH_PDL(mlstm_finish_kernel<T>, dim3(blocks), dim3(warps * 32), 0, stream, o, aux, (const T*)w, gate, ldg,
+                                         (T*)out, M, H, V, eps, gate_act));
+  JL_CUDA(cudaGetLastError());
+  return JL_OK;
+}
 
 extern "C" JL_API int jl_embed_pair_norm(const int* ids, const void* table, const void* pair, const void* norm_w, float* out,
                                          int* prev_tok, const int* cache_len, const int* pad_left, int B, int S, int W, int V,
@@ -270,7 +395,7 @@ extern "C" JL_API int jl_embed_pair_norm(const int* ids, const void* table, cons
   return JL_OK;
 }
 
-extern "C" JL_API int jl_causal_conv(const float* y, int ldy, int col0, int C, const void* w, const void* bias, float* state,
+extern "C" JL_API int jl_causal_conv(const float* y, int ldy, int col0, int C, const float* in_bias, const void* w, const void* bias, float* state,
                                      float* out, int ldo, const int* cache_len, const int* pad_left, int B, int S, int taps,
                                      int act, int dtype, void* stream) {
   JL_CHECK_ARG(B >= 1 && S >= 1 && C >= 1 && ldo >= C, "jl_causal_conv: bad shape");
@@ -278,8 +403,11 @@ extern "C" JL_API int jl_causal_conv(const float* y, int ldy, int col0, int C, c
   JL_CHECK_ARG(taps == 1 || state != nullptr, "jl_causal_conv: no state for %d taps", taps);
   const int chunk = CC_CHUNK;
   dim3 grid((C + 127) / 128, B, (S + chunk - 1) / chunk);
-  JL_DISPATCH_DTYPE(dtype, JL_LAUNCH_PDL(causal_conv_kernel<T>, dim3(grid), dim3(128), 0, stream, y, ldy, col0, C, (const T*)w,
-                                         (const T*)bias, state, out, ldo, cache_len, pad_left, S, taps, act, chunk));
+#define JL_CC(MT_)                                                                                                              \
+  JL_DISPATCH_DTYPE(dtype, JL_LAUNCH_PDL((causal_conv_kernel<T, MT_>), dim3(grid), dim3(128), 0, stream, y, ldy, col0, C, in_bias, \
+                                         (const T*)w, (const T*)bias, state, out, ldo, cache_len, pad_left, S, taps, act, chunk))
+  if (taps <= CC_FEW_TAPS) JL_CC(CC_FEW_TAPS); else JL_CC(CC_MAX_TAPS);
+#undef JL_CC
   JL_CUDA(cudaGetLastError());
   return JL_OK;
 }

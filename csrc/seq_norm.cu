@@ -191,6 +191,128 @@ __global__ void __launch_bounds__(256) branch_add_norm_kernel(const float* __res
   }
 }
 
+// Residual step of a block whose sublayers read the stream itself: with y = c1 * (y1 + bias) (+ c2 * y2),
+//     x[m, :] += y / sqrt(mean(y^2) + eps) * w;   h[m, :] = x[m, :] in the operand type (h == nullptr: the operands are x itself).
+// Vector path: the row stays in registers, 4 floats per thread and step, W <= THREADS * 4 * VPT; few rows take more threads.
+template <typename T, int VPT, int THREADS>
+__global__ void __launch_bounds__(THREADS) postnorm_cast_kernel(const float* __restrict__ y1, int ld1, const T* __restrict__ bias,
+                                                                float c1, const float* __restrict__ y2, int ld2, float c2,
+                                                                const T* __restrict__ w, float* __restrict__ x, T* __restrict__ h,
+                                                                int W, float eps, int vec) {
+  pdl_wait();                      // programmatic dependent launch: nothing is read before the predecessor is done
+  pdl_launch_dependents();
+  __shared__ float red[33];
+  const size_t m = blockIdx.x;
+  const float* a = y1 + m * ld1;
+  const float* b = y2 ? y2 + m * ld2 : nullptr;
+  float* xr = x + m * W;
+  float ss = 0.0f;
+  if (vec) {
+    const int nv = W / 4;
+    float yv[VPT][4], xv[VPT][4];
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int idx = threadIdx.x + i * THREADS;
+      if (idx < nv) {
+        float t[4];
+        load4(a + 4 * idx, yv[i]);
+        load4(xr + 4 * idx, xv[i]);
+        if (bias) {
+          load4(bias + 4 * idx, t);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) yv[i][j] += t[j];
+        }
+        if (b) {
+          load4(b + 4 * idx, t);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) yv[i][j] = c1 * yv[i][j] + c2 * t[j];
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) yv[i][j] *= c1;
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) ss += yv[i][j] * yv[i][j];
+      }
+    }
+    const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)W + eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int idx = threadIdx.x + i * THREADS;
+      if (idx < nv) {
+        float wv[4];
+        load4(w + 4 * idx, wv);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) xv[i][j] += yv[i][j] * r * wv[j];
+        store4(xr + 4 * idx, xv[i]);
+        if (h) store4(h + m * W + 4 * idx, xv[i]);
+      }
+    }
+    return;
+  }
+  auto value = [&](int i) {
+    const float v = c1 * (a[i] + (bias ? to_f(bias[i]) : 0.0f));
+    return b ? v + c2 * b[i] : v;
+  };
+  for (int i = threadIdx.x; i < W; i += THREADS) { const float v = value(i); ss += v * v; }
+  const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)W + eps);
+  for (int i = threadIdx.x; i < W; i += THREADS) {
+    const float v = xr[i] + value(i) * r * to_f(w[i]);
+    xr[i] = v;
+    if (h) h[m * W + i] = from_f<T>(v);
+  }
+}
+
+// out[m, :] = c1 * (y1[m, :] + bias) + c2 * y2[m, :]   (bias and y2 may be absent)
+template <typename T>
+__global__ void weighted_sum2_kernel(const float* __restrict__ y1, int ld1, const T* __restrict__ bias, float c1,
+                                     const float* __restrict__ y2, int ld2, float c2, float* __restrict__ out, int M, int W) {
+  pdl_wait();                      // programmatic dependent launch: nothing is read before the predecessor is done
+  pdl_launch_dependents();
+  const size_t total = (size_t)M * W;
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const size_t m = idx / W, i = idx % W;
+    const float v = c1 * (y1[m * ld1 + i] + (bias ? to_f(bias[i]) : 0.0f));
+    out[idx] = y2 ? v + c2 * y2[m * ld2 + i] : v;
+  }
+}
+
+// out[m, :] = o[m, :] / sqrt(mean(o^2) + eps) * w * act(gate[m, :]) over the WHOLE row (all heads together), one CTA per row
+template <typename T, int THREADS>
+__global__ void __launch_bounds__(THREADS) rownorm_gate_kernel(const float* __restrict__ o, const T* __restrict__ w,
+                                                               const float* __restrict__ gate, int ldg, T* __restrict__ out, int N,
+                                                               float eps, int gate_act, int vec) {
+  pdl_wait();                      // programmatic dependent launch: nothing is read before the predecessor is done
+  pdl_launch_dependents();
+  __shared__ float red[33];
+  const size_t m = blockIdx.x;
+  const float* orow = o + m * N;
+  const float* grow = gate + m * ldg;
+  float ss = 0.0f;
+  if (vec) {
+    for (int i = 4 * threadIdx.x; i < N; i += 4 * THREADS) {
+      float v[4];
+      load4(orow + i, v);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ss += v[j] * v[j];
+    }
+    const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)N + eps);
+    for (int i = 4 * threadIdx.x; i < N; i += 4 * THREADS) {
+      float v[4], wv[4], g[4];
+      load4(orow + i, v);
+      load4(w + i, wv);
+      load4(grow + i, g);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[j] = v[j] * r * wv[j] * apply_act(g[j], gate_act, 0.f, 0.f);
+      store4(out + m * N + i, v);
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < N; i += THREADS) { const float v = orow[i]; ss += v * v; }
+  const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)N + eps);
+  for (int i = threadIdx.x; i < N; i += THREADS)
+    out[m * N + i] = from_f<T>(orow[i] * r * to_f(w[i]) * apply_act(grow[i], gate_act, 0.f, 0.f));
+}
+
 // One warp per (token, head): out = o / sqrt(mean_v(o^2) + eps) * w[v] * act(gate)   (w == nullptr: no weight)
 template <typename T>
 __global__ void headnorm_gate_kernel(const float* __restrict__ o, const T* __restrict__ w, const float* __restrict__ gate,
@@ -313,6 +435,45 @@ extern "C" JL_API int jl_branch_add_norm(const float* y1, int ld1, const float* 
                                          mult, x, (const T*)w1, (T*)h1, (const T*)w2, (T*)h2, W, eps, (int)vec))
   if (vpt <= 1) JL_BA(1); else if (vpt <= 2) JL_BA(2); else if (vpt <= 4) JL_BA(4); else if (vpt <= 8) JL_BA(8); else JL_BA(16);
 #undef JL_BA
+  JL_CUDA(cudaGetLastError());
+  return JL_OK;
+}
+
+extern "C" JL_API int jl_postnorm_cast(const float* y1, int ld1, const void* bias, float c1, const float* y2, int ld2, float c2,
+                                       const void* w, float* x, void* h, int M, int W, float eps, int dtype, void* stream) {
+  JL_CHECK_ARG(M >= 1 && W >= 1 && y1 != nullptr && ld1 >= W && (y2 == nullptr || ld2 >= W), "jl_postnorm_cast: bad shape M=%d W=%d", M, W);
+  const int vec = W % 4 == 0 && ld1 % 4 == 0 && (y2 == nullptr || ld2 % 4 == 0) && W <= 256 * 4 * 16 &&
+                  ((uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)bias | (uintptr_t)w | (uintptr_t)x | (uintptr_t)h) % 16 == 0;
+#define JL_PC(V, TH)                                                                                                             \
+  JL_DISPATCH_DTYPE(dtype, JL_LAUNCH_PDL((postnorm_cast_kernel<T, V, TH>), dim3(M), dim3(TH), 0, (cudaStream_t)stream, y1, ld1,  \
+                                         (const T*)bias, c1, y2, ld2, c2, (const T*)w, x, (T*)h, W, eps, vec))
+  const int vpt = vec ? (W / 4 + 255) / 256 : 1;
+  if (vec && M <= 8 && vpt > 1 && vpt <= 8) { if (vpt <= 4) JL_PC(1, 1024); else JL_PC(2, 1024); }
+  else if (vpt <= 1) JL_PC(1, 256); else if (vpt <= 2) JL_PC(2, 256); else if (vpt <= 4) JL_PC(4, 256); else if (vpt <= 8) JL_PC(8, 256);
+  else JL_PC(16, 256);
+#undef JL_PC
+  JL_CUDA(cudaGetLastError());
+  return JL_OK;
+}
+
+extern "C" JL_API int jl_weighted_sum2(const float* y1, int ld1, const void* bias, float c1, const float* y2, int ld2, float c2,
+                                       float* out, int M, int W, int dtype, void* stream) {
+  JL_CHECK_ARG(M >= 1 && W >= 1 && y1 != nullptr && ld1 >= W && (y2 == nullptr || ld2 >= W), "jl_weighted_sum2: bad shape M=%d W=%d", M, W);
+  const size_t total = (size_t)M * W;
+  const int blocks = (int)((total + 255) / 256 < 148 * 8 ? (total + 255) / 256 : 148 * 8);
+  JL_DISPATCH_DTYPE(dtype, JL_LAUNCH_PDL(weighted_sum2_kernel<T>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, y1, ld1, (const T*)bias, c1,
+                                         y2, ld2, c2, out, M, W));
+  JL_CUDA(cudaGetLastError());
+  return JL_OK;
+}
+
+extern "C" JL_API int jl_rownorm_gate(const float* o, const void* w, const float* gate, int ldg, void* out, int M, int N, float eps,
+                                      int gate_act, int dtype, void* stream) {
+  JL_CHECK_ARG(M >= 1 && N >= 1 && ldg >= N && w != nullptr, "jl_rownorm_gate: bad shape M=%d N=%d", M, N);
+  JL_CHECK_ARG(gate_act >= 0 && gate_act <= ACT_LAST, "jl_rownorm_gate: bad activation %d", gate_act);
+  const int vec = N % 4 == 0 && ldg % 4 == 0 && ((uintptr_t)o | (uintptr_t)w | (uintptr_t)gate | (uintptr_t)out) % 16 == 0;
+  JL_DISPATCH_DTYPE(dtype, JL_LAUNCH_PDL((rownorm_gate_kernel<T, 256>), dim3(M), dim3(256), 0, (cudaStream_t)stream, o, (const T*)w, gate, ldg,
+                                         (T*)out, N, eps, gate_act, vec));
   JL_CUDA(cudaGetLastError());
   return JL_OK;
 }

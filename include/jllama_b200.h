@@ -385,9 +385,10 @@ int jl_embed_pair_norm(const int* ids, const void* table, const void* pair, cons
                        long long mul_cur, float eps, int dtype, void* stream);
 /* Causal convolution over time per channel: out[m, c] = act(bias[c] + sum_j w[c][taps-1-j] * in[token - j][c]), inputs fp32
  * columns col0 .. col0+C-1 of y, zeros before a sequence's start; state fp32 [B][taps-1][C] holds the last taps-1 inputs of
- * every row (read for the first tokens of the call, replaced by the call's last inputs).  w [C][taps], bias [C] or NULL. */
-int jl_causal_conv(const float* y, int ldy, int col0, int C, const void* w, const void* bias, float* state, float* out, int ldo,
-                   const int* cache_len, const int* pad_left, int B, int S, int taps, int act, int dtype, void* stream);
+ * every row (read for the first tokens of the call, replaced by the call's last inputs).  w [C][taps], bias [C] or NULL.
+ * in_bias fp32 [C] or NULL: added to every input (the projection's bias; the zeros before the start stay zero).  taps <= 32. */
+int jl_causal_conv(const float* y, int ldy, int col0, int C, const float* in_bias, const void* w, const void* bias, float* state,
+                   float* out, int ldo, const int* cache_len, const int* pad_left, int B, int S, int taps, int act, int dtype, void* stream);
 /* out[m] = c * (norm(a[m]) * wa + norm(b[m]) * wb), fp32 [M, W] (b NULL: one branch). */
 int jl_norm_mean2(const float* a, int lda, const void* wa, const float* b, int ldb, const void* wb, float c, float* out, int M,
                   int W, float eps, int dtype, void* stream);
@@ -449,21 +450,28 @@ int jl_attn_prep_ex(const float* y, int ldy, int q_off, int k_off, int v_off, vo
                     const int* cache_len, const int* pad_left, int B, int S, int H, int G, int D, int Dv, int T_cap,
                     const float* bias, int v_norm, int v_token_major, int dtype, void* stream);
 /* jl_attn_windowed with: gate (fp32 pre-activation of a sigmoid per head, column h of row m, pitch ldg; NULL: none); chunk > 0:
- * positions form blocks of `chunk` and a query sees the keys of its own block only; sink_logit fp32 [H]: the extra term of the
+ * positions form blocks of `chunk` and a query sees the keys of its own block only; softcap > 0: scores become softcap *
+ * tanh(score / softcap); sink_logit fp32 [H]: the extra term of the
  * denominator is exp(sink_logit[h]) (needs sink = 1; NULL: exp(0)); v_cos / v_sin: the cached values were rotated at their own
  * positions and every head's sum is rotated back by the query's position before the gate. */
 int jl_attn_masked(const void* q, const void* k_cache, const void* v_cache, void* out, const float* gate, int ldg,
                    const int* cache_len, const int* pad_left, int B, int S, int H, int G, int D, int Dv, int T_cap, int ldk, int ldv,
-                   long long k_bs, long long k_hs, long long v_bs, long long v_hs, int window, int chunk, float scale, float* scratch,
-                   int splits, int sink, const float* sink_logit, const float* v_cos, const float* v_sin, int v_max_pos,
+                   long long k_bs, long long k_hs, long long v_bs, long long v_hs, int window, int chunk, float scale, float softcap,
+                   float* scratch, int splits, int sink, const float* sink_logit, const float* v_cos, const float* v_sin, int v_max_pos,
                    int v_layout, float* out32, int dtype, void* stream);
 /* The tcgen05 prompt attention kernel (bfloat16, 128-wide heads; caches [B, nkv, T, 128]) with blocks of `chunk` positions, a sink in
  * the denominator (sink_logit fp32 [nh] or NULL for exp(0)), a sigmoid gate per (token, head) (fp32 pre-activation, pitch ldg) and the
  * turn back of values cached rotated at their own positions (v_cos / v_sin fp32 [v_max_pos][64], pairs m, m + 64).  `start`: slots
- * filled before this call's S tokens per row. */
+ * filled before this call's S tokens per row.  window > 0: a query sees itself and the window - 1 slots before it; softcap > 0: scores
+ * become softcap * tanh(score / softcap).  hd = 64 (without rotated values) runs jl_prefill_attn_mma_masked. */
 int jl_flash_prefill_masked(const void* q, const void* k_cache, const void* v_cache, const int* pad_left, void* out, int B, int S,
                             int nh, int nkv, int hd, int T, int start, float scale, int chunk, int sink, const float* sink_logit,
-                            const float* gate, int ldg, const float* v_cos, const float* v_sin, int v_max_pos, void* stream);
+                            const float* gate, int ldg, const float* v_cos, const float* v_sin, int v_max_pos, int window,
+                            float softcap, void* stream);
+/* jl_prefill_attn_mma (hd = 64) with the same options, values as they are. */
+int jl_prefill_attn_mma_masked(const void* q, const void* k_cache, const void* v_cache, const int* pad_left, void* out, int B, int S,
+                               int nh, int nkv, int hd, int T, int start, float scale, int window, int chunk, float softcap, int sink,
+                               const float* sink_logit, const float* gate, int ldg, void* stream);
 /* jl_moe_route with: choice_bias fp32 [E] added to the scores for the choice (group scores and top) only; experts n_real .. E-1
  * are identity experts: a chosen one is reported as expert -1 (jl_moe_sort and the grouped linears skip it) and its weight is
  * added to ident_w[m]. */
@@ -474,6 +482,42 @@ int jl_moe_route_ex(const float* z, int ldz, int M, int E, int top, int groups, 
 int jl_moe_combine_ex(const float* z, int ldz, const int* pos, const float* wt, int top, const float* shared, int lds,
                       const float* gate, int ldg, float* out, int M, int W, const int* idx, const float* ident_w, const void* x,
                       int ldx, int dtype, void* stream);
+
+/* ---- sublayers that read the stream itself, q / k norms over all heads, mixed values, activated linear attention, matrix memory
+ *      with exponential gates (csrc/seq_norm.cu, attn_generic.cu, gla_scan.cu, seq_mix.cu) */
+
+/* With y = c1 * (y1 + bias) + c2 * y2 (bias [W] of dtype or NULL, y2 or NULL; y1, y2 fp32 [M, W] with row pitches): x[m] += y / rms(y) * w
+ * in place (fp32), and h[m] = the updated row in dtype (h NULL: not wanted). */
+int jl_postnorm_cast(const float* y1, int ld1, const void* bias, float c1, const float* y2, int ld2, float c2, const void* w, float* x,
+                     void* h, int M, int W, float eps, int dtype, void* stream);
+/* out[m] = c1 * (y1[m] + bias) + c2 * y2[m], fp32 [M, W]; bias [W] of dtype and y2 may be NULL. */
+int jl_weighted_sum2(const float* y1, int ld1, const void* bias, float c1, const float* y2, int ld2, float c2, float* out, int M, int W,
+                     int dtype, void* stream);
+/* out[m] = o[m] / rms(o[m]) * w * act(gate[m]) over whole rows of N columns; o fp32 [M, N]; gate fp32 with row pitch ldg; w, out of dtype. */
+int jl_rownorm_gate(const float* o, const void* w, const float* gate, int ldg, void* out, int M, int N, float eps, int gate_act, int dtype,
+                    void* stream);
+/* q / k rows (H*D and G*D columns of y) RMS-normed as a whole with the weights q_norm_w [H*D] / k_norm_w [G*D], rotated (`rot` leading
+ * channels of every head, pairs as layout), q to q_out [B*S, H, D], k and v appended to caches [B][G][T_cap][D] / [..][Dv].  bias: fp32,
+ * indexed like the columns of y.  v_first fp32 [B*S, G*Dv] (pitch ldvf) with the scalar *v_lambda of dtype: v <- (1 - l) v + l v_first. */
+int jl_attn_prep_all(const float* y, int ldy, int q_off, int k_off, int v_off, void* q_out, void* k_cache, void* v_cache,
+                     const float* cos_t, const float* sin_t, int max_pos, int rot, int layout, const void* q_norm_w,
+                     const void* k_norm_w, float eps, const int* cache_len, const int* pad_left, int B, int S, int H, int G, int D,
+                     int Dv, int T_cap, const float* bias, const float* v_first, int ldvf, const void* v_lambda, int dtype,
+                     void* stream);
+/* jl_retention_scan without rotation and scales over projections that pass an activation (q, k and v alike). */
+int jl_activated_scan(const float* y, int ldy, int q_off, int k_off, int v_off, const float* head_decay, int act, float* state, float* o,
+                      const int* cache_len, const int* pad_left, int B, int S, int H, int D, int Dv, float* ws, void* stream);
+/* Log gates i = cap tanh((y[i_off + h] + i_bias[h]) / cap), f = logsigmoid(cap tanh((y[f_off + h] + f_bias[h]) / cap)), running maximum
+ * m = max(f + m, i) (m_state fp32 [B][H], read and replaced); aux fp32 [B*S][3H]: exp(f + m_before - m) | exp(i - m) | exp(-m). */
+int jl_mlstm_gates(const float* y, int ldy, int i_off, int f_off, const void* i_bias, const void* f_bias, float cap, float* m_state,
+                   float* aux, const int* cache_len, const int* pad_left, int B, int S, int H, int dtype, void* stream);
+/* S_t = aux[h] S_(t-1) + aux[H + h] k_t [v_t | 1]^T, o_t = S_t^T (q_scale q_t); state fp32 [B][H][D][Dv + 1], o fp32 [B*S][H][Dv + 1] (last
+ * column: n . q); ws: jl_gla_scan_ws_floats(B, S, H, D, Dv + 1) floats for prompts, NULL for a few tokens. */
+int jl_mlstm_scan(const float* y, int ldy, int q_off, int k_off, int v_off, const float* aux, int ld_aux, float q_scale, float* state,
+                  float* o, const int* cache_len, const int* pad_left, int B, int S, int H, int D, int Dv, float* ws, void* stream);
+/* v = o[.., :V] / (max(|o[.., V]|, aux[2H + h]) + 1e-6); out[m, h] = v / rms(v) * w[h*V ..] * act(gate[m, h*V ..]). */
+int jl_mlstm_finish(const float* o, const float* aux, const void* w, const float* gate, int ldg, void* out, int M, int H, int V,
+                    float eps, int gate_act, int dtype, void* stream);
 
 #ifdef __cplusplus
 }

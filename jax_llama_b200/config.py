@@ -16,7 +16,7 @@ import json
 import logging
 import os
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Union
 
 logger = logging.getLogger(__name__)
 
@@ -254,21 +254,35 @@ class RotaryScaling:
 
 
 @dataclass
+class WavelengthScaling:
+    """Frequency interpolation by wavelength: waves longer than original / low positions are slowed by `factor`, waves
+    shorter than original / high are kept; in between the two frequencies are blended in proportion to the number of waves
+    that fit into `original`."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+
+@dataclass
 class RotarySpec:
     """Rotary embedding on the first `dims` channels of each head, frequencies base^(-2i/dims).  layout "interleaved"
     pairs channel 2i with 2i+1, "half" pairs channel i with i + dims/2."""
     dims: int
     base: float
     layout: str = "interleaved"
-    scaling: Optional[RotaryScaling] = None
+    scaling: Optional[Union[RotaryScaling, WavelengthScaling]] = None
 
     @staticmethod
     def parse(rot: Optional[Dict[str, Any]], layout: str = "interleaved") -> Optional["RotarySpec"]:
         if not rot:
             return None
         sc = rot.get("scaling")
-        scaling = None
-        if sc:
+        scaling: Any = None
+        if sc and "low" in sc:
+            scaling = WavelengthScaling(factor=float(sc["factor"]), low=float(sc["low"]), high=float(sc["high"]),
+                                        original=float(sc["original"]))
+        elif sc:
             scaling = RotaryScaling(factor=float(sc["factor"]), original=float(sc["original"]), fast=float(sc["fast"]),
                                     slow=float(sc["slow"]))
         return RotarySpec(int(rot["dims"]), float(rot["base"]), layout, scaling)
@@ -298,6 +312,14 @@ class AttentionMixerSpec:
     sink_learned: bool = False      # the sink's logit is `sink` [heads] instead of 0 (needs sink)
     v_rot: bool = False             # values are rotated at their own position over all vdim channels (frequencies rot.base^(-2m/vdim),
                                     # the pairing of rot.layout, no interpolation), every head's sum is rotated back at the query's
+    qk_norm_all: bool = False       # RMS norm over all channels of q (and of k) together, weights `q.norm` / `k.norm` of that size,
+                                    # BEFORE the rotation
+    softcap: float = 0.0            # > 0: scores become softcap · tanh(score / softcap) before the softmax
+    conv: int = 0                   # > 0: q and k pass a causal convolution of `conv` taps (`q.conv`, `k.conv`) right after the
+                                    # projection and its bias
+    v_from_k: bool = False          # no value projection: the values are the keys before norm and rotation
+    v_mix: str = ""                 # "first": this layer's values are kept for the step; "mix": v <- (1 - vmix) v + vmix v_first
+    out_bias: bool = False          # the output projection has a bias (`o.b`)
     kind: str = "attention"
 
 
@@ -370,12 +392,39 @@ class DeltaMixerSpec:
 
 
 @dataclass
+class LightningMixerSpec:
+    """Linear attention with one fixed decay per head over silu-activated q, k and v: S_t = decay_h S_(t-1) + k_t v_tᵀ,
+    o_t = S_tᵀ q_t; the concatenated heads RMS-normed together with the weight `norm`, gated by sigmoid."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: List[float] = field(default_factory=list)
+    kind: str = "lightning"
+
+
+@dataclass
+class MlstmMixerSpec:
+    """Matrix memory with an exponential input gate: log gates i = cap tanh((i + i.b) / cap), f = logsigmoid(cap tanh((f + f.b) /
+    cap)) per head, running maximum m_t = max(f + m_(t-1), i) from 0, S_t = exp(f + m_(t-1) - m_t) S_(t-1) + exp(i - m_t) k vᵀ,
+    n_t the same with k alone, o = S_tᵀ q / (max(|n_t · q|, exp(-m_t)) + 1e-6); q scaled by dim^(-1/2); read-out divided by its
+    RMS per head, times `norm` (all heads), gated by sigmoid."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+    kind: str = "mlstm"
+
+
+@dataclass
 class ParallelMixerSpec:
-    """Two mixers side by side on the same input; each result is RMS-normed over the model width with its own weight and
-    the mixer returns `scale` times their sum."""
+    """Two mixers side by side on the same input.  combine "norm": each result is RMS-normed over the model width with its own
+    weight and the mixer returns `scale` times their sum; "weighted": left_scale · left + right_scale · right."""
     left: Any
     right: Any
     scale: float = 0.5
+    combine: str = "norm"
+    left_scale: float = 1.0
+    right_scale: float = 1.0
     kind: str = "parallel"
 
 
@@ -439,7 +488,8 @@ class HybridConfig:
 
     * ``block``: "sandwich" — mixer and feed-forward one after the other, each between a norm before and a norm after,
       x += norm(sublayer(norm(x))); "parallel" — both read norms of the same x, x += residual_mult · (mixer + ff);
-      "parallel_shared" — the same with ONE norm that both sublayers read;
+      "parallel_shared" — the same with ONE norm that both sublayers read; "post" — one after the other, reading the stream
+      itself, each normed on the way back only, x += norm(sublayer(x));
     * ``tied_head``: the logits are taken against the embedding table (no ``head`` tensor); ``embed_norm``: a norm
       (``embed.norm``) right after the embedding;
     * ``norm_offset``: what is added to a stored norm weight (1 for weights stored around zero);
@@ -816,3 +866,81 @@ class DatozenConfig(HybridConfig):
                 raise ValueError(f"layer {i}: top {f.top} of {n} experts")
             if f.groups > 1 and (n % f.groups or not 1 <= f.keep <= f.groups or f.keep * (n // f.groups) < f.top):
                 raise ValueError(f"layer {i}: {f.groups} groups (keep {f.keep}) cannot give {f.top} of {n} experts")
+
+
+class KetolixConfig(HybridConfig):
+    """Ketolix: a decoder whose sublayers read the residual stream itself and are normed on the way back only — ``x += norm1
+    (mixer(x)); x += norm2(ff(x))`` — with logits against the embedding table.
+
+    Mixers: "attention" — grouped heads; q and k normed over all their channels together; interleaved rotary embedding with
+    wavelength-interpolated frequencies; scores capped by tanh; sliding window; a learned logit per head in the softmax
+    denominator; values mixed with the values of the first layer that mixes.  "parallel" — weighted sum of softmax attention
+    whose q and k pass a short causal convolution (values are the convolved keys, biases on q, k and the output, a sigmoid gate per
+    head) and linear attention with fixed decays over silu-activated q, k, v.  "mlstm" — matrix memory with an exponential
+    input gate.  Feed-forward: a silu-gated dense layer.
+
+    ``config.json``: ``vocab``, ``width``, ``norm.eps`` and ``layers[i]`` = ``{type, mixer, mlp}`` with, for "attention",
+    ``mixer.{heads, kv_heads, dim, vdim, scale, softcap, v_mix, mask.size, rot.{dims, base, scaling.{factor, low, high,
+    original}}}``; for "parallel", ``mixer.{left_scale, right_scale}``, ``mixer.left.{heads, kv_heads, dim, vdim, scale, conv,
+    mask.size, rot.{dims, base}}`` and ``mixer.right.{heads, dim, vdim, decay}``; for "mlstm", ``mixer.{heads, dim, vdim,
+    gate_cap}``; ``mlp`` null or ``{kind: dense, ff}``."""
+
+    model_type = "ketolix"
+    architecture = "Ketolix"
+    block = "post"
+    norm_offset = 0.0
+    tied_head = True
+
+    def _parse_mixer(self, i: int, d: Dict[str, Any]) -> Any:
+        m = d["mixer"]
+        kind = d["type"]
+        if kind == "attention":
+            mixing = [j for j, l in enumerate(self.layer_dicts) if l["type"] == "attention" and l["mixer"].get("v_mix")]
+            v_mix = "" if i not in mixing else ("first" if i == mixing[0] else "mix")
+            return AttentionMixerSpec(**self._attention_sizes(m), qk_unit_norm=False, head_gate=False, qk_norm_all=True, sink=True,
+                                      sink_learned=True, softcap=float(m.get("softcap") or 0.0), v_mix=v_mix)
+        if kind == "parallel":
+            a, r = m["left"], m["right"]
+            left = AttentionMixerSpec(**self._attention_sizes(a), qk_unit_norm=False, head_gate=True, bias=True, out_bias=True,
+                                      qk_norm_all=True, conv=int(a.get("conv") or 0), v_from_k=True)
+            right = LightningMixerSpec(heads=int(r["heads"]), dim=int(r["dim"]), vdim=int(r["vdim"]),
+                                       decay=[float(v) for v in r["decay"]])
+            return ParallelMixerSpec(left=left, right=right, combine="weighted", left_scale=float(m["left_scale"]),
+                                     right_scale=float(m["right_scale"]))
+        if kind == "mlstm":
+            return MlstmMixerSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), gate_cap=float(m["gate_cap"]))
+        raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+
+    @staticmethod
+    def _attention_sizes(m: Dict[str, Any]) -> Dict[str, Any]:
+        return dict(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads", m["heads"])), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                    scale=float(m["scale"]), rot=RotarySpec.parse(m.get("rot"), "interleaved"), kv_from=None,
+                    window=int((m.get("mask") or {}).get("size") or 0))
+
+    def _parse_mlp(self, i: int, mlp: Optional[Dict[str, Any]]) -> Any:
+        if mlp is None:
+            return None
+        if mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+        return DenseMlpSpec(ff=int(mlp["ff"]), act="silu", gated=True)
+
+    def _validate_layer(self, i: int, l: HybridLayerSpec) -> None:
+        m = l.mixer
+        for a in ([m] if m.kind == "attention" else [m.left] if m.kind == "parallel" else []):
+            if min(a.heads, a.kv_heads, a.dim, a.vdim) <= 0 or a.heads % a.kv_heads or a.window < 0 or a.softcap < 0:
+                raise ValueError(f"layer {i}: attention sizes heads {a.heads}, kv_heads {a.kv_heads}, window {a.window}")
+            if a.rot is not None and (a.rot.dims % 2 or a.rot.dims > a.dim):
+                raise ValueError(f"layer {i}: rot.dims {a.rot.dims} must be even and at most dim {a.dim}")
+            if a.v_from_k and a.vdim != a.dim:
+                raise ValueError(f"layer {i}: values that are the keys have vdim {a.vdim} = dim {a.dim}")
+            if a.v_mix == "mix":
+                first = next(s.mixer for s in self.layers if getattr(s.mixer, "v_mix", "") == "first")
+                if (first.kv_heads, first.vdim) != (a.kv_heads, a.vdim):
+                    raise ValueError(f"layer {i}: value sizes differ from the first layer that mixes")
+        if m.kind == "parallel":
+            if m.left.conv < 0:
+                raise ValueError(f"layer {i}: {m.left.conv} taps")
+            if len(m.right.decay) != m.right.heads:
+                raise ValueError(f"layer {i}: {len(m.right.decay)} decays for {m.right.heads} heads")
+        if m.kind == "mlstm" and m.gate_cap <= 0:
+            raise ValueError(f"layer {i}: gate_cap must be positive")

@@ -7,8 +7,9 @@ token-at-a-time stream are inherited; what changes is
 
 * the weights (per-layer mixers from `models/mixers.py`, feed-forwards from `models/feedforward.py`; norm weights
   stored around zero or plain, as the configuration says),
-* the block form: sublayers one after the other, each between two norms ("sandwich"), or mixer and feed-forward
-  side by side on two norms of the same stream, their scaled sum added to it ("parallel"),
+* the block form: sublayers one after the other, each between two norms ("sandwich") or reading the stream itself and normed on the
+  way back only ("post"), or mixer and feed-forward side by side on two norms of the same stream, their scaled sum added to it
+  ("parallel"),
 * the cache: per attention layer a key / value cache with that layer's head sizes (none for a layer that reads another
   layer's), per recurrent layer an fp32 state, all advanced by the same device-side fill level and left-pad counts; a
   stretch of layers that runs several times over with the same weights (`config.loop`) has one cache entry per layer RUN,
@@ -19,7 +20,7 @@ token-at-a-time stream are inherited; what changes is
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import astuple, dataclass, field
 from typing import Any, Dict, List, Optional, Tuple
 
 import torch
@@ -45,6 +46,7 @@ class HybridCache(DeviceKVCache):
     states: List[Any] = field(default_factory=list)      # per layer: fp32 tensor(s) carried from token to token
     length: int = 0
     prev_tok: Optional[torch.Tensor] = None              # int32 [B]: every row's last token (embeddings that hash token pairs)
+    step_values: dict = field(default_factory=dict)      # what a layer leaves for later layers of the same step (fp32 views)
     step_ids: Optional[torch.Tensor] = None              # int32 [B·S]: the tokens of the step in flight (per-layer token inputs)
 
     @property
@@ -202,12 +204,13 @@ class HybridEngine(B200Engine):
         self.mega_max_batch = 0
         self.eps = float(config.rms_norm_eps)
         self.norm_offset = float(config.norm_offset)          # 1: norm weights are stored around zero
-        if config.block not in ("sandwich", "parallel", "parallel_shared"):
+        if config.block not in ("sandwich", "parallel", "parallel_shared", "post"):
             raise ValueError(f"unknown block form {config.block!r}")
         self.parallel = config.block in ("parallel", "parallel_shared")
         self.shared_norm = config.block == "parallel_shared"      # one norm per block, read by both sublayers
-        if self.parallel and self.norm_offset != 0.0:
-            raise ValueError("parallel blocks take plain norm weights")
+        self.post = config.block == "post"                        # sublayers read the stream itself, their results are normed
+        if (self.parallel or self.post) and self.norm_offset != 0.0:
+            raise ValueError("parallel and post-norm blocks take plain norm weights")
         present = {name: tuple(t.shape) for name, t in tensors.items()}
         rank = next((int(t.shape[0]) for name, t in tensors.items() if name.endswith("mix.a1")), 16)
         want = tensor_shapes(config, decay_rank=rank, present=present)
@@ -244,12 +247,12 @@ class HybridEngine(B200Engine):
             p = f"l{i}."
             w = {k[len(p) + 4:]: get(k) for k in want if k.startswith(p + "mix.")}
             layer = HybridLayer(mixer=MIXERS[l.mixer.kind](l.mixer, w, self.eps), norm1=get(p + "norm1"))
-            if not self.parallel:
+            if config.block == "sandwich":
                 layer.norm1b = get(p + "norm1b")
             if l.mlp is not None:
                 if not self.shared_norm:
                     layer.norm2 = get(p + "norm2")
-                if not self.parallel:
+                if config.block == "sandwich":
                     layer.norm2b = get(p + "norm2b")
                 fw = {k[len(p) + 4:]: get(k) for k in want if k.startswith(p + "mlp.")}
                 try:
@@ -299,7 +302,7 @@ class HybridEngine(B200Engine):
             key: Tuple = (2, 1.0, None)
         else:
             sc = rot.scaling
-            key = (int(rot.dims), float(rot.base), None if sc is None else (sc.factor, sc.original, sc.fast, sc.slow))
+            key = (int(rot.dims), float(rot.base), None if sc is None else (type(sc).__name__, *astuple(sc)))
         have = self._rope.get(key)
         if have is None or (rot is not None and have[0].shape[0] < length):
             if torch.cuda.is_current_stream_capturing():
@@ -309,7 +312,11 @@ class HybridEngine(B200Engine):
         return have
 
     def _ropes(self, mixer: Any, length: int) -> Tuple[torch.Tensor, ...]:
-        """The tables a mixer's `forward` gets: cos / sin of its q / k rotation, then those of its value rotation if it has one."""
+        """The tables a mixer's `forward` gets: cos / sin of its q / k rotation, then those of its value rotation if it has one;
+        a mixer made of several gets one such tuple per side."""
+        sides = getattr(mixer, "sides", None)
+        if sides is not None:
+            return tuple(self._ropes(m, length) for m in sides)
         rope = self._rope_for(getattr(mixer.spec, "rot", None), length)
         vrot = getattr(mixer, "value_rot", None)
         return rope if vrot is None else rope + self._rope_for(vrot, length)
@@ -324,8 +331,7 @@ class HybridEngine(B200Engine):
         if self.pos_table is not None and max_length - 1 > self.pos_table.shape[0]:
             raise ValueError(f"max_length {max_length} exceeds the {self.pos_table.shape[0]} learned positions")
         for l in self.layers:
-            if getattr(l.mixer.spec, "rot", None) is not None:
-                self._ropes(l.mixer, max_length)
+            self._ropes(l.mixer, max_length)
 
     # ------------------------------------------------------------------ cache
     def new_cache(self, batch: int, max_length: int) -> HybridCache:
@@ -386,6 +392,8 @@ class HybridEngine(B200Engine):
             raise NotImplementedError("explicit position_ids are not supported by the hybrid engine (left padding is)")
         if self.parallel:
             return self._layers_parallel(x, B, S, cache)
+        if self.post:
+            return self._layers_post(x, B, S, cache)
         eps, off = self.eps, self.norm_offset
         stack = [self.layers[i] for i in self.runs]
         n = len(stack)
@@ -401,6 +409,21 @@ class HybridEngine(B200Engine):
                 h = SK.postnorm_add(z, l.norm2b, x, eps, off, w_next=nxt)
             if self.capture_streams is not None:
                 self.capture_streams.append(x.clone())
+        return x
+
+    def _layers_post(self, x: torch.Tensor, B: int, S: int, cache: HybridCache) -> torch.Tensor:
+        """Sublayers that read the stream itself: x += norm1(mixer(x)); x += norm2(ff(x)).  One kernel per sublayer sums the mixer's
+        parts, norms the sum, adds it and leaves the stream in the operand type for the next sublayer (true float32: the stream)."""
+        h = x if self.dtype == torch.float32 else SK.act_cast(x, self.dtype)
+        for i, li in enumerate(self.runs):
+            l = self.layers[li]
+            p = l.mixer.parts(h, B, S, cache, i, self._ropes(l.mixer, cache.capacity))
+            h = SK.postnorm_cast(p.y1, l.norm1, x, self.eps, bias=p.bias, c1=p.c1, y2=p.y2, c2=p.c2)
+            if l.ff is not None:
+                h = SK.postnorm_cast(l.ff.run(h), l.norm2, x, self.eps)
+            if self.capture_streams is not None:
+                self.capture_streams.append(x.clone())
+        cache.step_values.clear()
         return x
 
     def _layers_parallel(self, x: torch.Tensor, B: int, S: int, cache: HybridCache) -> torch.Tensor:
@@ -495,11 +518,13 @@ def random_tensors(config: Any, device: Any = "cuda", seed: int = 0, decay_rank:
         return torch.randn(shape, generator=g, device=dev, dtype=torch.float32)
 
     for name, shape in tensor_shapes(config, decay_rank).items():
-        if name.endswith("mix.norm") or (config.norm_offset == 0.0 and len(shape) == 1 and "norm" in name):
+        if name.endswith("mix.norm") or name.endswith("right.norm") or (config.norm_offset == 0.0 and len(shape) == 1 and "norm" in name):
             t = 1.0 + 0.1 * randn(shape)
         elif name.endswith("mix.a2.b"):
             t = 2.0 + 2.0 * randn(shape)
-        elif len(shape) == 1:
+        elif name.endswith("mix.f.b"):                       # forget gates that keep from a few to hundreds of tokens
+            t = 3.0 + 2.0 * randn(shape)
+        elif len(shape) <= 1:
             t = 0.1 * randn(shape)
         elif name == "embed":
             t = randn(shape)

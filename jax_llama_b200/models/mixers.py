@@ -12,12 +12,12 @@ The output projection, the norms around the sublayer and the residual sum belong
 from __future__ import annotations
 
 import math
-from typing import Dict, List, Optional, Tuple
+from typing import Dict, List, NamedTuple, Optional, Tuple
 
 import torch
 
-from ..config import (AttentionMixerSpec, DeltaMixerSpec, GlaMixerSpec, LatentAttentionMixerSpec, ParallelMixerSpec,
-                      RetentionMixerSpec, RotaryScaling, RotarySpec, StateSpaceMixerSpec)
+from ..config import (AttentionMixerSpec, DeltaMixerSpec, GlaMixerSpec, LatentAttentionMixerSpec, LightningMixerSpec, MlstmMixerSpec,
+                      ParallelMixerSpec, RetentionMixerSpec, RotaryScaling, RotarySpec, StateSpaceMixerSpec, WavelengthScaling)
 from ..ops import _lib
 from ..ops import kernels as K
 from ..ops import seq_kernels as SK
@@ -36,14 +36,23 @@ def _stack_rows(parts: List[torch.Tensor], multiple: int = 8) -> Tuple[torch.Ten
     return torch.cat(parts, 0).contiguous(), offs
 
 
-def rotary_frequencies(dims: int, base: float, scaling: Optional[RotaryScaling] = None) -> Tuple[torch.Tensor, float]:
-    """float64 frequencies base^(-2i/dims), i < dims/2, and the factor on cos / sin.  With `scaling`: the channel index
+def rotary_frequencies(dims: int, base: float, scaling: "Optional[RotaryScaling | WavelengthScaling]" = None
+                       ) -> Tuple[torch.Tensor, float]:
+    """float64 frequencies base^(-2i/dims), i < dims/2, and the factor on cos / sin.  With a `WavelengthScaling`: wavelength
+    2π / f above original / low: divided by `factor`; below original / high: kept; else blended by (original / wavelength − low) /
+    (high − low).  With a `RotaryScaling`: the channel index
     at which `original` positions make t turns is n(t) = dims · ln(original / (2π t)) / (2 ln base); channels below
     floor(n(fast)) keep their frequency, channels above ceil(n(slow)) are divided by `factor`, linear ramp between."""
     i = torch.arange(dims // 2, dtype=torch.float64)
     freq = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / dims)
     if scaling is None:
         return freq, 1.0
+    if isinstance(scaling, WavelengthScaling):
+        wl = 2.0 * math.pi / freq
+        s = (scaling.original / wl - scaling.low) / (scaling.high - scaling.low if scaling.high != scaling.low else 1.0)
+        mid = (1.0 - s) * freq / scaling.factor + s * freq
+        out = torch.where(wl < scaling.original / scaling.high, freq, mid)
+        return torch.where(wl > scaling.original / scaling.low, freq / scaling.factor, out), 1.0
 
     def channel_of(turns: float) -> float:
         return dims * math.log(scaling.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
@@ -54,8 +63,8 @@ def rotary_frequencies(dims: int, base: float, scaling: Optional[RotaryScaling] 
     return freq / scaling.factor * ramp + freq * (1.0 - ramp), 0.1 * math.log(scaling.factor) + 1.0
 
 
-def rotary_table(dims: int, base: float, length: int, device: torch.device, scaling: Optional[RotaryScaling] = None
-                 ) -> Tuple[torch.Tensor, torch.Tensor]:
+def rotary_table(dims: int, base: float, length: int, device: torch.device,
+                 scaling: "Optional[RotaryScaling | WavelengthScaling]" = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """cos / sin of position · frequency for the dims/2 channel pairs, as fp32 [length, dims/2] (angles formed in
     float64; the scaling's factor on cos / sin is in the table)."""
     freq, mult = rotary_frequencies(dims, base, scaling)
@@ -64,15 +73,30 @@ def rotary_table(dims: int, base: float, length: int, device: torch.device, scal
             (torch.sin(ang) * mult).float().to(device).contiguous())
 
 
+class MixerParts(NamedTuple):
+    """A mixer's contribution c1 · (y1 + bias) + c2 · y2 before it is summed, for layer stacks that sum it in their residual step."""
+    y1: torch.Tensor
+    bias: Optional[torch.Tensor] = None
+    c1: float = 1.0
+    y2: Optional[torch.Tensor] = None
+    c2: float = 0.0
+
+
 class Mixer:
-    """What the layer stack asks of a mixer.  `run` gives the input of the output projection `wo`; `forward` the mixer's
-    fp32 contribution [M, width] (a mixer made of several overrides it).  `shapes(spec, W, rank_of)` lists the checkpoint
+    """What the layer stack asks of a mixer.  `run` gives the input of the output projection `wo`; `parts` the terms of the mixer's
+    contribution, `forward` their fp32 sum [M, width] (a mixer made of several overrides them).  `shapes(spec, W, rank_of)` lists the checkpoint
     tensors under the mixer's prefix; `rank_of(name, default)` is the first dimension the checkpoint gives a tensor whose
     inner size no configuration key fixes."""
 
     def forward(self, h: torch.Tensor, B: int, S: int, cache: "object", layer: int, rope: Optional[Tuple] = None
                 ) -> torch.Tensor:
-        return SK.linear(self.run(h, B, S, cache, layer, rope), self.wo)
+        p = self.parts(h, B, S, cache, layer, rope)
+        return p.y1 if p.bias is None and p.y2 is None and p.c1 == 1.0 else SK.weighted_sum2(*p)
+
+    def parts(self, h: torch.Tensor, B: int, S: int, cache: "object", layer: int, rope: Optional[Tuple] = None) -> MixerParts:
+        return MixerParts(SK.linear(self.run(h, B, S, cache, layer, rope), self.wo), bias=self.out_bias)
+
+    out_bias: Optional[torch.Tensor] = None        # bias of the output projection
 
 
 class _CacheView:
@@ -104,17 +128,22 @@ class AttentionMixer(Mixer):
     either pairing of the rotated channels (`rot.layout`), values rotated at their own position and the head's sum rotated back
     at the query's (`v_rot`: the value cache holds rotated values, so a cached value never has to be touched again and the
     weighted sum depends on relative positions only), blocks of `chunk` positions instead of (or besides) a window, and a
-    learned sink logit per head.  These run the masked form of the generic attention kernels."""
+    learned sink logit per head.  These run the masked form of the generic attention kernels.
+
+    And: an RMS norm over all heads of q (of k) together (`qk_norm_all`); scores capped by tanh (`softcap`); a causal convolution on q
+    and k behind the projection (`conv`, its last inputs are state), values that are the convolved keys (`v_from_k`); values mixed
+    with those of the first such layer (`v_mix`: that layer leaves a view of its fp32 values with the cache for the step, the
+    mixed value is what later layers cache); a bias on the output projection (`out_bias`)."""
 
     kind = "attention"
 
     def __init__(self, spec: AttentionMixerSpec, w: Dict[str, torch.Tensor], eps: float):
         self.spec, self.eps = spec, float(eps)
         self.shares_kv = spec.kv_from is not None
-        parts = [w["q"]] + ([] if self.shares_kv else [w["k"], w["v"]]) + ([w["g"]] if spec.head_gate else [])
-        self.w_in, offs = _stack_rows(parts)
+        own = [] if self.shares_kv else [w["k"]] if spec.v_from_k else [w["k"], w["v"]]
+        self.w_in, offs = _stack_rows([w["q"]] + own + ([w["g"]] if spec.head_gate else []))
         self.q_off = offs[0]
-        self.k_off, self.v_off = (-1, -1) if self.shares_kv else (offs[1], offs[2])
+        self.k_off, self.v_off = (-1, -1) if self.shares_kv else (offs[1], offs[1] if spec.v_from_k else offs[2])
         self.g_off = offs[-1] if spec.head_gate else -1
         self.wo = w["o"].contiguous()
         self.dtype = self.wo.dtype
@@ -123,15 +152,26 @@ class AttentionMixer(Mixer):
         if spec.bias:                                      # fp32 over the columns of the stacked projection
             self.bias = torch.zeros(self.w_in.shape[0], dtype=torch.float32, device=self.wo.device)
             for name, off in (("q", self.q_off), ("k", self.k_off), ("v", self.v_off)):
-                if off >= 0:
+                if off >= 0 and name + ".b" in w:
                     self.bias[off:off + w[name].shape[0]] = w[name + ".b"].float()
         self.talk = w["talk"].contiguous() if spec.talking_heads else None
         if spec.talking_heads and (self.shares_kv or spec.head_gate):
             raise ValueError("mixed attention weights go with a layer's own keys / values and no head gate")
         self.plain = not (spec.bias or spec.v_unit_norm or spec.window or spec.sink or spec.talking_heads or spec.qk_norm
-                          or spec.chunk or spec.v_rot or (spec.rot is not None and spec.rot.layout != "interleaved"))
-        self.q_norm = w["q.norm"].contiguous() if spec.qk_norm else None
-        self.k_norm = w["k.norm"].contiguous() if spec.qk_norm and not self.shares_kv else None
+                          or spec.chunk or spec.v_rot or spec.softcap or spec.qk_norm_all or spec.conv or spec.v_from_k
+                          or (spec.rot is not None and spec.rot.layout != "interleaved"))
+        any_norm = spec.qk_norm or spec.qk_norm_all
+        self.q_norm = w["q.norm"].contiguous() if any_norm else None
+        self.k_norm = w["k.norm"].contiguous() if any_norm and not self.shares_kv else None
+        self.conv_w = torch.cat([w["q.conv"], w["k.conv"]], 0).contiguous() if spec.conv else None
+        self.v_lambda = w["vmix"].contiguous() if spec.v_mix == "mix" else None
+        self.out_bias = w["o.b"].contiguous() if spec.out_bias else None
+        if (spec.conv or spec.v_from_k or spec.v_mix) and not spec.qk_norm_all:
+            raise ValueError("convolved keys and mixed values go with norms over all heads")
+        if spec.qk_norm_all and (spec.qk_norm or spec.qk_unit_norm or self.shares_kv or spec.talking_heads or spec.v_unit_norm or spec.v_rot):
+            raise ValueError("norms over all heads do not combine with per-head norms, shared keys, mixed heads or rotated values")
+        if spec.v_from_k and spec.dim != spec.vdim:
+            raise ValueError("values that are the keys have the keys' size")
         self.sink_logit = w["sink"].float().contiguous() if spec.sink_learned else None
         if spec.sink_learned and not spec.sink:
             raise ValueError("a learned sink logit needs the sink")
@@ -144,9 +184,17 @@ class AttentionMixer(Mixer):
     def shapes(spec: AttentionMixerSpec, W: int, rank_of: "object" = None) -> Dict[str, Tuple[int, ...]]:
         out: Dict[str, Tuple[int, ...]] = {"q": (spec.heads * spec.dim, W), "o": (W, spec.heads * spec.vdim)}
         if spec.kv_from is None:
-            out["k"], out["v"] = (spec.kv_heads * spec.dim, W), (spec.kv_heads * spec.vdim, W)
+            out["k"] = (spec.kv_heads * spec.dim, W)
+            if not spec.v_from_k:
+                out["v"] = (spec.kv_heads * spec.vdim, W)
         if spec.head_gate:
             out["g"] = (spec.heads, W)
+        if spec.conv:
+            out["q.conv"], out["k.conv"] = (spec.heads * spec.dim, spec.conv), (spec.kv_heads * spec.dim, spec.conv)
+        if spec.v_mix:
+            out["vmix"] = ()
+        if spec.out_bias:
+            out["o.b"] = (W,)
         if spec.bias:
             for n in ("q", "k", "v"):
                 if n in out:
@@ -157,12 +205,15 @@ class AttentionMixer(Mixer):
             out["q.norm"] = (spec.dim,)
             if spec.kv_from is None:
                 out["k.norm"] = (spec.dim,)
+        if spec.qk_norm_all:
+            out["q.norm"], out["k.norm"] = (spec.heads * spec.dim,), (spec.kv_heads * spec.dim,)
         if spec.sink_learned:
             out["sink"] = (spec.heads,)
         return out
 
     def weights(self) -> List[torch.Tensor]:
-        return [self.w_in, self.wo] + [t for t in (self.talk, self.q_norm, self.k_norm, self.sink_logit) if t is not None]
+        return [self.w_in, self.wo] + [t for t in (self.talk, self.q_norm, self.k_norm, self.sink_logit, self.conv_w, self.v_lambda,
+                                                   self.out_bias) if t is not None]
 
     def new_cache(self, batch: int, length: int, device: torch.device) -> Optional[Tuple[torch.Tensor, torch.Tensor]]:
         if self.shares_kv:
@@ -175,7 +226,33 @@ class AttentionMixer(Mixer):
                 torch.zeros((batch, s.kv_heads, length, s.vdim), dtype=self.dtype, device=device))
 
     def new_state(self, batch: int, device: torch.device) -> Optional[torch.Tensor]:
+        s = self.spec
+        if s.conv > 1:                                     # the last conv - 1 projected q | k of every row
+            return torch.zeros((batch, s.conv - 1, (s.heads + s.kv_heads) * s.dim), dtype=torch.float32, device=device)
         return None
+
+    def _prepare_all(self, y: torch.Tensor, q: torch.Tensor, kc: torch.Tensor, vc: torch.Tensor, rope: Tuple[torch.Tensor, torch.Tensor],
+                     rot: int, layout: int, B: int, S: int, cache: "object", layer: int) -> None:
+        """Convolution, norms over all heads, rotation, mixed values and the append, for the designs that have them."""
+        s = self.spec
+        src, q_off, k_off, v_off, bias = y, self.q_off, self.k_off, self.v_off, self.bias
+        if s.conv:
+            n = self.conv_w.shape[0]                                  # q | k are the leading columns of the stacked projection
+            src = SK.causal_conv(y, q_off, self.conv_w, None, cache.states[layer], cache.len_dev, cache.pad_left, B, S,
+                                 act=SK.ACT_NONE, in_bias=bias[:n] if bias is not None else None)
+            if not s.v_from_k:
+                raise NotImplementedError("a convolution on q and k beside a value projection")
+            q_off, k_off, v_off, bias = 0, s.heads * s.dim, s.heads * s.dim, None
+        v_first = None
+        if s.v_mix == "first":
+            if self.bias is not None:
+                raise NotImplementedError("mixed values with a bias")
+            cache.step_values["first"] = y[:, v_off:v_off + s.kv_heads * s.vdim]
+        elif s.v_mix == "mix":
+            v_first = cache.step_values["first"]
+        SK.attn_prep_all(src, q_off, k_off, v_off, q, kc, vc, rope[0], rope[1], rot, layout, self.q_norm, self.k_norm, self.eps,
+                         cache.len_dev, cache.pad_left, B, S, s.heads, s.kv_heads, s.dim, s.vdim, bias=bias, v_first=v_first,
+                         v_lambda=self.v_lambda)
 
     def run(self, h: torch.Tensor, B: int, S: int, cache: "object", layer: int, rope: Tuple[torch.Tensor, torch.Tensor]
             ) -> torch.Tensor:
@@ -187,28 +264,32 @@ class AttentionMixer(Mixer):
         rot = s.rot.dims if s.rot is not None else 0
         layout = SK.ROT_LAYOUTS[s.rot.layout] if s.rot is not None else 0
         v_cos, v_sin = (rope[2], rope[3]) if s.v_rot else (None, None)      # the engine appends the tables of `value_rot`
-        SK.attn_prep(y, self.q_off, self.k_off, self.v_off, q, None if self.shares_kv else kc,
-                     None if self.shares_kv else vc, rope[0], rope[1], rot, s.qk_unit_norm, self.eps, cache.len_dev,
-                     cache.pad_left, B, S, s.heads, s.kv_heads, s.dim, s.vdim, bias=self.bias, v_unit_norm=s.v_unit_norm,
-                     v_token_major=s.talking_heads, layout=layout, q_norm_w=self.q_norm,
-                     k_norm_w=self.k_norm if self.k_norm is not None else self.q_norm, v_cos=v_cos, v_sin=v_sin)
+        if s.qk_norm_all:
+            self._prepare_all(y, q, kc, vc, rope, rot, layout, B, S, cache, layer)
+        else:
+            SK.attn_prep(y, self.q_off, self.k_off, self.v_off, q, None if self.shares_kv else kc,
+                         None if self.shares_kv else vc, rope[0], rope[1], rot, s.qk_unit_norm, self.eps, cache.len_dev,
+                         cache.pad_left, B, S, s.heads, s.kv_heads, s.dim, s.vdim, bias=self.bias, v_unit_norm=s.v_unit_norm,
+                         v_token_major=s.talking_heads, layout=layout, q_norm_w=self.q_norm,
+                         k_norm_w=self.k_norm if self.k_norm is not None else self.q_norm, v_cos=v_cos, v_sin=v_sin)
         if s.talking_heads:
             return self._attend_mixed(q, kc, vc, cache, B, S)
         gate = y[:, self.g_off:self.g_off + s.heads] if s.head_gate else None
-        if not self.plain and (gate is not None or s.chunk or s.sink_learned or s.v_rot):
+        if not self.plain and (gate is not None or s.chunk or s.sink_learned or s.v_rot or s.softcap):
             if S > 1 and self._flash_masked_shape():
-                # prompts of 128-wide heads in bfloat16: the tcgen05 kernel with the block bound, the sink, the gate and the turn
-                # back in its softmax and epilogue
+                # prompts of 128-wide heads in bfloat16: the tcgen05 kernel with the block bound, the window, the cap, the sink, the
+                # gate and the turn back in its softmax and epilogue; 64-wide heads: the warp-level kernel
                 out = torch.empty((B * S, s.heads * s.vdim), dtype=self.dtype, device=q.device)
                 _lib.check(_lib.lib().jl_flash_prefill_masked(
                     q.data_ptr(), kc.data_ptr(), vc.data_ptr(), cache.pad_left.data_ptr(), out.data_ptr(), B, S, s.heads,
                     s.kv_heads, s.dim, kc.shape[2], int(cache.index), float(s.scale), int(s.chunk), int(s.sink),
                     K._p(self.sink_logit), K._p(gate), gate.stride(0) if gate is not None else 0, K._p(v_cos), K._p(v_sin),
-                    v_cos.shape[0] if v_cos is not None else 0, K._stream()), "jl_flash_prefill_masked")
+                    v_cos.shape[0] if v_cos is not None else 0, int(s.window), float(s.softcap), K._stream()),
+                    "jl_flash_prefill_masked")
                 return out
             return SK.attn_masked(q, kc, vc, cache.len_dev, cache.pad_left, B, S, s.heads, s.kv_heads, s.dim, s.vdim, s.scale,
                                   gate=gate, window=s.window, chunk=s.chunk, sink=s.sink, sink_logit=self.sink_logit,
-                                  v_cos=v_cos, v_sin=v_sin, v_layout=layout)
+                                  v_cos=v_cos, v_sin=v_sin, v_layout=layout, softcap=s.softcap)
         if not self.plain:
             T = kc.shape[2]
             return SK.attn_windowed(q, kc, vc, cache.len_dev, cache.pad_left, B, S, s.heads, s.kv_heads, s.dim, s.vdim, T,
@@ -242,12 +323,12 @@ class AttentionMixer(Mixer):
         return out
 
     def _flash_masked_shape(self) -> bool:
-        """Whether prompts can run the tcgen05 kernel in its masked form: bfloat16, 128-wide keys and values, a layer's own
-        head-major caches, no window, values rotated in the half-split pairing (or not at all)."""
+        """Whether prompts can run the tensor-core kernels in their masked form: bfloat16, 128-wide (or 64-wide, values not rotated)
+        keys and values, a layer's own head-major caches, values rotated in the half-split pairing (or not at all)."""
         s = self.spec
-        return (SK.tensor_cores_enabled() and self.dtype == torch.bfloat16 and s.dim == s.vdim == 128 and not self.shares_kv
-                and s.heads // s.kv_heads in (1, 2, 4, 8, 16) and not (s.window or s.bias or s.v_unit_norm or s.talking_heads)
-                and (not s.v_rot or s.rot.layout == "half") and _lib.has("jl_flash_prefill_masked"))
+        return (SK.tensor_cores_enabled() and self.dtype == torch.bfloat16 and s.dim == s.vdim and not self.shares_kv
+                and (s.dim == 128 or (s.dim == 64 and not s.v_rot)) and not s.talking_heads
+                and s.heads // s.kv_heads in (1, 2, 4, 8, 16) and (not s.v_rot or s.rot.layout == "half") and _lib.has("jl_flash_prefill_masked"))
 
     def _library_shape(self) -> bool:
         s = self.spec
@@ -551,7 +632,8 @@ class DeltaRuleMixer(Mixer):
 
 class ParallelMixer(Mixer):
     """Two mixers side by side on the same input: scale · (norm(left(h)) · w_left + norm(right(h)) · w_right), the norms
-    over the model width.  Each side keeps its own cache / state; the layer's cache entries are pairs."""
+    over the model width, or (combine "weighted") left_scale · left(h) + right_scale · right(h), summed in the residual step of the
+    stacks that take a mixer's parts.  Each side keeps its own cache / state; the layer's cache entries are pairs."""
 
     kind = "parallel"
 
@@ -561,8 +643,8 @@ class ParallelMixer(Mixer):
         for side, sub in (("left", spec.left), ("right", spec.right)):
             sw = {k[len(side) + 1:]: v for k, v in w.items() if k.startswith(side + ".") and k != side + ".out"}
             self.sides.append(MIXERS[sub.kind](sub, sw, eps))
-        self.out_norms = [w["left.out"].contiguous(), w["right.out"].contiguous()]
-        self.dtype = self.out_norms[0].dtype
+        self.out_norms = [w["left.out"].contiguous(), w["right.out"].contiguous()] if spec.combine == "norm" else []
+        self.dtype = self.sides[0].dtype
 
     @staticmethod
     def shapes(spec: ParallelMixerSpec, W: int, rank_of: "object" = None) -> Dict[str, Tuple[int, ...]]:
@@ -571,7 +653,8 @@ class ParallelMixer(Mixer):
             sub_rank = (lambda name, default, side=side: rank_of(side + "." + name, default)) if rank_of else None
             for name, shape in MIXERS[sub.kind].shapes(sub, W, sub_rank).items():
                 out[f"{side}.{name}"] = shape
-            out[f"{side}.out"] = (W,)
+            if spec.combine == "norm":
+                out[f"{side}.out"] = (W,)
         return out
 
     def weights(self) -> List[torch.Tensor]:
@@ -589,8 +672,15 @@ class ParallelMixer(Mixer):
 
     OVERLAP_ROWS = 8               # up to this many rows the two sides run on two streams
 
-    def forward(self, h: torch.Tensor, B: int, S: int, cache: "object", layer: int, rope: Optional[Tuple] = None
-                ) -> torch.Tensor:
+    def parts(self, h: torch.Tensor, B: int, S: int, cache: "object", layer: int, rope: Optional[Tuple] = None) -> MixerParts:
+        s = self.spec
+        if s.combine == "norm":
+            left, right = self._both(h, B, S, cache, layer, rope)
+            return MixerParts(SK.norm_mean2(left.y1, self.out_norms[0], right.y1, self.out_norms[1], s.scale, self.eps))
+        left, right = self._both(h, B, S, cache, layer, rope)
+        return MixerParts(left.y1, left.bias, s.left_scale, right.y1, s.right_scale)
+
+    def _both(self, h: torch.Tensor, B: int, S: int, cache: "object", layer: int, rope: Optional[Tuple]) -> Tuple[MixerParts, MixerParts]:
         """With a few rows (decoding) neither side fills the GPU and each is a chain of short dependent kernels, so the right
         side runs on a second stream beside the left one (inside a graph capture the fork and join become edges of the
         captured graph).  Prompts stay on one stream: their tensor-core GEMMs share one split-K workspace."""
@@ -602,17 +692,109 @@ class ParallelMixer(Mixer):
             self._fork.record(main)
             self._side.wait_event(self._fork)
             with torch.cuda.stream(self._side):
-                right = self.sides[1].forward(h, B, S, views[1], layer, rope)
+                right = self.sides[1].parts(h, B, S, views[1], layer, self._rope_of(1, rope))
                 self._join.record(self._side)
-            left = self.sides[0].forward(h, B, S, views[0], layer, rope)
+            left = self.sides[0].parts(h, B, S, views[0], layer, self._rope_of(0, rope))
             main.wait_event(self._join)
         else:
-            left = self.sides[0].forward(h, B, S, views[0], layer, rope)
-            right = self.sides[1].forward(h, B, S, views[1], layer, rope)
-        return SK.norm_mean2(left, self.out_norms[0], right, self.out_norms[1], self.spec.scale, self.eps)
+            left = self.sides[0].parts(h, B, S, views[0], layer, self._rope_of(0, rope))
+            right = self.sides[1].parts(h, B, S, views[1], layer, self._rope_of(1, rope))
+        for p in (left, right) if self.out_norms else (right,):
+            if p.bias is not None or p.y2 is not None:
+                raise NotImplementedError("an output bias on this side of a parallel mixer")
+        return left, right
+
+    @staticmethod
+    def _rope_of(side: int, rope: Optional[Tuple]) -> Optional[Tuple]:
+        """The engine hands a mixer made of several one tuple of tables per side."""
+        return rope[side] if rope is not None and isinstance(rope[0], tuple) else rope
+
+
+class LightningMixer(Mixer):
+    """Linear attention with one fixed decay per head over silu-activated projections (see `LightningMixerSpec`): the scan kernels of
+    gated linear attention with the activation applied where q, k and v are read; one norm over all heads' read-outs, weight and
+    sigmoid gate in one pass."""
+
+    kind = "lightning"
+
+    def __init__(self, spec: LightningMixerSpec, w: Dict[str, torch.Tensor], eps: float):
+        self.spec, self.eps = spec, float(eps)
+        self.w_in, offs = _stack_rows([w["q"], w["k"], w["v"], w["g"]])
+        self.q_off, self.k_off, self.v_off, self.g_off = offs
+        self.norm = w["norm"].contiguous()
+        self.wo = w["o"].contiguous()
+        self.dtype = self.wo.dtype
+        self.decay = torch.tensor([float(a) for a in spec.decay], dtype=torch.float64).to(torch.float32).to(self.wo.device)
+
+    @staticmethod
+    def shapes(spec: LightningMixerSpec, W: int, rank_of: "object" = None) -> Dict[str, Tuple[int, ...]]:
+        nk, nv = spec.heads * spec.dim, spec.heads * spec.vdim
+        return {"q": (nk, W), "k": (nk, W), "v": (nv, W), "g": (nv, W), "o": (W, nv), "norm": (nv,)}
+
+    def weights(self) -> List[torch.Tensor]:
+        return [self.w_in, self.norm, self.wo]
+
+    def new_cache(self, batch: int, length: int, device: torch.device) -> None:
+        return None
+
+    def new_state(self, batch: int, device: torch.device) -> torch.Tensor:
+        s = self.spec
+        return torch.zeros((batch, s.heads, s.dim, s.vdim), dtype=torch.float32, device=device)
+
+    def run(self, h: torch.Tensor, B: int, S: int, cache: "object", layer: int, rope: Optional[Tuple] = None) -> torch.Tensor:
+        s = self.spec
+        y = SK.linear(h, self.w_in)                                   # fp32 [M, q | k | v | gate]
+        o = SK.activated_scan(y, self.q_off, self.k_off, self.v_off, self.decay, SK.ACT_SILU, cache.states[layer], cache.len_dev,
+                              cache.pad_left, B, S, s.heads, s.dim, s.vdim)
+        return SK.rownorm_gate(o, self.norm, y[:, self.g_off:self.g_off + s.heads * s.vdim], self.eps, SK.ACT_SIGMOID)
+
+
+class MlstmMixer(Mixer):
+    """Matrix memory with exponential gates (see `MlstmMixerSpec`).  One stacked projection [q | k | v | gate | i | f]; a small kernel
+    turns the gate columns into a decay, an input scale and a denominator floor per (token, head), the running maximum found by a
+    max-plus scan over time; then the scan kernels of gated linear attention, the normaliser n being one more value column
+    (constantly one), and a finishing pass: division, per-head norm, weight, sigmoid gate."""
+
+    kind = "mlstm"
+
+    def __init__(self, spec: MlstmMixerSpec, w: Dict[str, torch.Tensor], eps: float):
+        self.spec, self.eps = spec, float(eps)
+        self.w_in, offs = _stack_rows([w["q"], w["k"], w["v"], w["g"], w["i"], w["f"]])
+        self.q_off, self.k_off, self.v_off, self.g_off, self.i_off, self.f_off = offs
+        self.i_bias, self.f_bias = w["i.b"].contiguous(), w["f.b"].contiguous()
+        self.norm = w["norm"].contiguous()
+        self.wo = w["o"].contiguous()
+        self.dtype = self.wo.dtype
+
+    @staticmethod
+    def shapes(spec: MlstmMixerSpec, W: int, rank_of: "object" = None) -> Dict[str, Tuple[int, ...]]:
+        nk, nv, H = spec.heads * spec.dim, spec.heads * spec.vdim, spec.heads
+        return {"q": (nk, W), "k": (nk, W), "v": (nv, W), "g": (nv, W), "o": (W, nv), "norm": (nv,), "i": (H, W), "i.b": (H,),
+                "f": (H, W), "f.b": (H,)}
+
+    def weights(self) -> List[torch.Tensor]:
+        return [self.w_in, self.i_bias, self.f_bias, self.norm, self.wo]
+
+    def new_cache(self, batch: int, length: int, device: torch.device) -> None:
+        return None
+
+    def new_state(self, batch: int, device: torch.device) -> Tuple[torch.Tensor, torch.Tensor]:
+        """The memory with its normaliser as the last column, and the running maximum (which starts at 0)."""
+        s = self.spec
+        return (torch.zeros((batch, s.heads, s.dim, s.vdim + 1), dtype=torch.float32, device=device),
+                torch.zeros((batch, s.heads), dtype=torch.float32, device=device))
+
+    def run(self, h: torch.Tensor, B: int, S: int, cache: "object", layer: int, rope: Optional[Tuple] = None) -> torch.Tensor:
+        s = self.spec
+        state, m_state = cache.states[layer]
+        y = SK.linear(h, self.w_in)                                   # fp32 [M, q | k | v | gate | i | f]
+        o, aux = SK.mlstm_scan(y, self.q_off, self.k_off, self.v_off, self.i_off, self.f_off, self.i_bias, self.f_bias, s.gate_cap,
+                               s.dim ** -0.5, state, m_state, cache.len_dev, cache.pad_left, B, S, s.heads, s.dim, s.vdim)
+        return SK.mlstm_finish(o, aux, self.norm, y[:, self.g_off:self.g_off + s.heads * s.vdim], s.heads, s.vdim, self.eps,
+                               SK.ACT_SIGMOID)
 
 
 MIXERS = {"attention": AttentionMixer, "gla": GlaMixer, "latent_attention": LatentAttentionMixer,
           "retention": RetentionMixer, "state_space": StateSpaceMixer, "channel_delta": DeltaRuleMixer,
-          "parallel": ParallelMixer}
+          "parallel": ParallelMixer, "lightning": LightningMixer, "mlstm": MlstmMixer}
 

@@ -83,7 +83,7 @@ _HYBRID = {
     "jl_gemm_grouped": (i32, [vp, vp, vp, i32, i32, i32, i32, ip, ip, i32, i32, vp]),
     "jl_moe_combine": (i32, [fp, i32, ip, fp, i32, fp, i32, fp, i32, fp, i32, i32, vp]),
     "jl_embed_pair_norm": (i32, [ip, vp, vp, vp, fp, ip, ip, ip] + [i32] * 5 + [i64, i64, f32, i32, vp]),
-    "jl_causal_conv": (i32, [fp, i32, i32, i32, vp, vp, fp, fp, i32, ip, ip] + [i32] * 5 + [vp]),
+    "jl_causal_conv": (i32, [fp, i32, i32, i32, fp, vp, vp, fp, fp, i32, ip, ip] + [i32] * 5 + [vp]),
     "jl_norm_mean2": (i32, [fp, i32, vp, fp, i32, vp, f32, fp, i32, i32, f32, i32, vp]),
     "jl_gated_groupnorm": (i32, [fp, fp, i32, vp, i32, fp, i32, vp, vp, i32, i32, i32, f32, i32, i32, vp]),
     "jl_glu_act": (i32, [fp, i32, i32, i32, vp, i32, i32, i32, i32, i32, f32, f32, ip, i32, i32, vp]),
@@ -97,10 +97,19 @@ _HYBRID = {
     "jl_side_gate_rows": (i32, [fp, i32, ip, vp, i32, i32, vp, vp, i32, i32, i32, i32, i32, i32, vp]),
     "jl_attn_prep_ex": (i32, [fp, i32, i32, i32, i32, vp, vp, vp, fp, fp, i32, i32, i32, i32, vp, vp, f32, fp, fp, i32, i32, ip, ip]
                         + [i32] * 7 + [fp, i32, i32, i32, vp]),
-    "jl_attn_masked": (i32, [vp, vp, vp, vp, fp, i32, ip, ip] + [i32] * 9 + [i64] * 4 + [i32, i32, f32, fp, i32, i32, fp, fp, fp,
+    "jl_attn_masked": (i32, [vp, vp, vp, vp, fp, i32, ip, ip] + [i32] * 9 + [i64] * 4 + [i32, i32, f32, f32, fp, i32, i32, fp, fp, fp,
                                                                                       i32, i32, fp, i32, vp]),
     "jl_moe_route_ex": (i32, [fp] + [i32] * 9 + [f32, fp, fp, i32, fp, ip, fp, vp]),
     "jl_moe_combine_ex": (i32, [fp, i32, ip, fp, i32, fp, i32, fp, i32, fp, i32, i32, ip, fp, vp, i32, i32, vp]),
+    "jl_postnorm_cast": (i32, [fp, i32, vp, f32, fp, i32, f32, vp, fp, vp, i32, i32, f32, i32, vp]),
+    "jl_weighted_sum2": (i32, [fp, i32, vp, f32, fp, i32, f32, fp, i32, i32, i32, vp]),
+    "jl_rownorm_gate": (i32, [fp, vp, fp, i32, vp, i32, i32, f32, i32, i32, vp]),
+    "jl_attn_prep_all": (i32, [fp, i32, i32, i32, i32, vp, vp, vp, fp, fp, i32, i32, i32, vp, vp, f32, ip, ip] + [i32] * 7
+                         + [fp, fp, i32, vp, i32, vp]),
+    "jl_activated_scan": (i32, [fp, i32, i32, i32, i32, fp, i32, fp, fp, ip, ip] + [i32] * 5 + [fp, vp]),
+    "jl_mlstm_gates": (i32, [fp, i32, i32, i32, vp, vp, f32, fp, fp, ip, ip] + [i32] * 4 + [vp]),
+    "jl_mlstm_scan": (i32, [fp, i32, i32, i32, i32, fp, i32, f32, fp, fp, ip, ip] + [i32] * 5 + [fp, vp]),
+    "jl_mlstm_finish": (i32, [fp, fp, vp, fp, i32, vp, i32, i32, i32, f32, i32, i32, vp]),
     "jl_delta_scan": (i32, [fp, i32, i32, i32, i32, i32, fp, i32, i32, i32, vp, vp, vp, fp, fp, ip, ip] + [i32] * 6 + [fp, i32, vp]),
 }
 
@@ -108,7 +117,8 @@ _OPTIONAL = {
     "jl_flash_prefill_occupancy": (i32, [i32]),
     "jl_decode_mega_stages": (i32, [i32, i32, i32, i32, i32, i32]),
     "jl_flash_prefill": (i32, [vp, vp, vp, ip, ip, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp]),
-    "jl_flash_prefill_masked": (i32, [vp, vp, vp, ip, vp] + [i32] * 7 + [f32, i32, i32, fp, fp, i32, fp, fp, i32, vp]),
+    "jl_flash_prefill_masked": (i32, [vp, vp, vp, ip, vp] + [i32] * 7 + [f32, i32, i32, fp, fp, i32, fp, fp, i32, i32, f32, vp]),
+    "jl_prefill_attn_mma_masked": (i32, [vp, vp, vp, ip, vp] + [i32] * 7 + [f32, i32, i32, f32, i32, fp, fp, i32, vp]),
     "jl_prefill_attn_mma": (i32, [vp, vp, vp, ip, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp]),
 }
 

@@ -38,6 +38,9 @@ SUBSETS = {
     "hybrid_attention": ["error.cu", "seq_norm.cu", "seq_linear.cu", "attn_generic.cu", "moe.cu", "seq_mix.cu", "seq_token.cu",
                          "sample_full.cu", "gemm_tcgen05.cu", "gemm_2cta.cu", "tensormap.cu", "flash_prefill.cu",
                          "prefill_attn_mma.cu"],
+    # softmax attention (masked forms) and linear scans: no experts, no delta rule, no per-token inputs
+    "hybrid_scan": ["error.cu", "seq_norm.cu", "seq_linear.cu", "attn_generic.cu", "gla_scan.cu", "seq_mix.cu", "sample_full.cu",
+                    "gemm_tcgen05.cu", "gemm_2cta.cu", "tensormap.cu", "flash_prefill.cu", "prefill_attn_mma.cu"],
 }
 
 

@@ -337,10 +337,11 @@ def attn_masked(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, c
                 pad_left: Optional[torch.Tensor], B: int, S: int, H: int, G: int, D: int, Dv: int, scale: float, *,
                 gate: Optional[torch.Tensor] = None, window: int = 0, chunk: int = 0, sink: bool = False,
                 sink_logit: Optional[torch.Tensor] = None, v_cos: Optional[torch.Tensor] = None,
-                v_sin: Optional[torch.Tensor] = None, v_layout: int = 0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                v_sin: Optional[torch.Tensor] = None, v_layout: int = 0, out: Optional[torch.Tensor] = None, softcap: float = 0.0
+                ) -> torch.Tensor:
     """Causal attention of S new tokens per row over caches [B, G, T, D] / [B, G, T, Dv] with everything the kernels take:
     gate fp32 view [M, H] (sigmoid per head on the output); window; chunk > 0: positions form blocks of `chunk` and a query sees
-    the keys of its own block only; sink with an optional learned logit per head (fp32 [H]); v_cos / v_sin fp32
+    the keys of its own block only; softcap > 0: scores become softcap · tanh(score / softcap); sink with an optional learned logit per head (fp32 [H]); v_cos / v_sin fp32
     [positions, Dv/2]: the values were cached rotated at their own positions and every head's sum is rotated back by the
     query's position, before the gate."""
     T_cap = k_cache.shape[2]
@@ -357,7 +358,7 @@ def attn_masked(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, c
             scratch = torch.empty(B * H * splits * (Dv + 2), dtype=torch.float32, device=q.device)
     _lib.check(L.jl_attn_masked(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), _p(gate), gate.stride(0) if gate is not None else 0,
-        _p(cache_len), _p(pad_left), B, S, H, G, D, Dv, T_cap, D, Dv, 0, 0, 0, 0, int(window), int(chunk), float(scale), _p(scratch),
+        _p(cache_len), _p(pad_left), B, S, H, G, D, Dv, T_cap, D, Dv, 0, 0, 0, 0, int(window), int(chunk), float(scale), float(softcap), _p(scratch),
         splits, int(sink), _p(sink_logit), _p(v_cos), _p(v_sin), v_cos.shape[0] if v_cos is not None else 0, int(v_layout), 0,
         dtype_code(q.dtype), _stream()), "jl_attn_masked")
     return out
@@ -494,15 +495,18 @@ def embed_pair_norm(ids: torch.Tensor, table: torch.Tensor, pair: torch.Tensor, 
 
 def causal_conv(y: torch.Tensor, col0: int, w: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor],
                 cache_len: Optional[torch.Tensor], pad_left: Optional[torch.Tensor], B: int, S: int, act: int = ACT_SILU,
-                out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                out: Optional[torch.Tensor] = None, in_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """act(causal convolution over time) of the C = w.shape[0] columns of y (fp32) from col0; w [C, taps], the last tap on the
-    current token; state fp32 [B, taps-1, C]: the inputs before this call, replaced by this call's last."""
+    current token; state fp32 [B, taps-1, C]: the inputs before this call, replaced by this call's last.  in_bias fp32 [C]: part
+    of every input (not of the zeros before a sequence's start)."""
     _need(y, torch.float32, "y")
+    if in_bias is not None:
+        _need(in_bias, torch.float32, "in_bias")
     C, taps = w.shape
     if out is None:
         out = torch.empty((B * S, C), dtype=torch.float32, device=y.device)
-    _lib.check(_lib.lib().jl_causal_conv(y.data_ptr(), y.stride(0), int(col0), C, w.data_ptr(), _p(bias), _p(state), out.data_ptr(),
-                                         out.stride(0), _p(cache_len), _p(pad_left), B, S, taps, act, dtype_code(w.dtype), _stream()),
+    _lib.check(_lib.lib().jl_causal_conv(y.data_ptr(), y.stride(0), int(col0), C, _p(in_bias), w.data_ptr(), _p(bias), _p(state),
+                                         out.data_ptr(), out.stride(0), _p(cache_len), _p(pad_left), B, S, taps, act, dtype_code(w.dtype), _stream()),
                "jl_causal_conv")
     return out
 
@@ -646,3 +650,115 @@ def branch_add_cast(x: torch.Tensor, y1: Optional[torch.Tensor], y2: Optional[to
                                              y2.stride(0) if y2 is not None else 0, float(mult), x.data_ptr(), xc.data_ptr(), M, W,
                                              dtype_code(dtype), _stream()), "jl_branch_add_cast")
     return xc
+
+
+# --------------------------------------------------------------------------- sublayers on the stream itself, norms over all heads, matrix memory
+def postnorm_cast(y1: torch.Tensor, w: torch.Tensor, x: torch.Tensor, eps: float, *, bias: Optional[torch.Tensor] = None, c1: float = 1.0,
+                  y2: Optional[torch.Tensor] = None, c2: float = 0.0) -> torch.Tensor:
+    """x += norm(c1 · (y1 + bias) + c2 · y2) · w in place (fp32); returns the updated rows in w's dtype (x itself for fp32)."""
+    _need(y1, torch.float32, "y1")
+    _need(x, torch.float32, "x")
+    if y2 is not None:
+        _need(y2, torch.float32, "y2")
+    M, W = x.shape
+    h = torch.empty((M, W), dtype=w.dtype, device=x.device) if w.dtype != torch.float32 else None
+    _lib.check(_lib.lib().jl_postnorm_cast(y1.data_ptr(), y1.stride(0), _p(bias), float(c1), _p(y2), y2.stride(0) if y2 is not None else 0,
+                                           float(c2), w.data_ptr(), x.data_ptr(), _p(h), M, W, float(eps), dtype_code(w.dtype),
+                                           _stream()), "jl_postnorm_cast")
+    return h if h is not None else x
+
+
+def weighted_sum2(y1: torch.Tensor, bias: Optional[torch.Tensor], c1: float, y2: Optional[torch.Tensor], c2: float) -> torch.Tensor:
+    """c1 · (y1 + bias) + c2 · y2, fp32 [M, W]."""
+    _need(y1, torch.float32, "y1")
+    M, W = y1.shape
+    out = torch.empty((M, W), dtype=torch.float32, device=y1.device)
+    _lib.check(_lib.lib().jl_weighted_sum2(y1.data_ptr(), y1.stride(0), _p(bias), float(c1), _p(y2), y2.stride(0) if y2 is not None else 0,
+                                           float(c2), out.data_ptr(), M, W, dtype_code(bias.dtype) if bias is not None else 1,
+                                           _stream()), "jl_weighted_sum2")
+    return out
+
+
+def rownorm_gate(o: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, eps: float, gate_act: int = ACT_SIGMOID) -> torch.Tensor:
+    """o fp32 [M, N] → norm over the whole row · w · act(gate) in w's dtype; gate: fp32 view [M, N]."""
+    _need(o, torch.float32, "o")
+    _need(gate, torch.float32, "gate")
+    M, N = o.shape
+    out = torch.empty((M, N), dtype=w.dtype, device=o.device)
+    _lib.check(_lib.lib().jl_rownorm_gate(o.data_ptr(), w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), M, N, float(eps),
+                                          gate_act, dtype_code(w.dtype), _stream()), "jl_rownorm_gate")
+    return out
+
+
+def attn_prep_all(y: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                  cos: torch.Tensor, sin: torch.Tensor, rot: int, layout: int, q_norm_w: torch.Tensor, k_norm_w: torch.Tensor, eps: float,
+                  cache_len: torch.Tensor, pad_left: Optional[torch.Tensor], B: int, S: int, H: int, G: int, D: int, Dv: int, *,
+                  bias: Optional[torch.Tensor] = None, v_first: Optional[torch.Tensor] = None, v_lambda: Optional[torch.Tensor] = None
+                  ) -> None:
+    """Norm q and k over all their heads together (weights [H·D] / [G·D]), rotate, append k, v to the caches [B, G, T, D] /
+    [B, G, T, Dv].  bias: fp32 over the columns of y.  v_first fp32 view [B·S, G·Dv] with the scalar v_lambda: values become
+    (1 − λ) v + λ v_first."""
+    _need(y, torch.float32, "y")
+    if bias is not None:
+        _need(bias, torch.float32, "bias")
+    if v_first is not None:
+        _need(v_first, torch.float32, "v_first")
+    _lib.check(_lib.lib().jl_attn_prep_all(
+        y.data_ptr(), y.stride(0), q_off, k_off, v_off, q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), cos.data_ptr(),
+        sin.data_ptr(), cos.shape[0], rot, int(layout), q_norm_w.data_ptr(), k_norm_w.data_ptr(), float(eps), _p(cache_len), _p(pad_left),
+        B, S, H, G, D, Dv, k_cache.shape[2], _p(bias), _p(v_first), v_first.stride(0) if v_first is not None else 0, _p(v_lambda),
+        dtype_code(q_out.dtype), _stream()), "jl_attn_prep_all")
+
+
+def activated_scan(y: torch.Tensor, q_off: int, k_off: int, v_off: int, head_decay: torch.Tensor, act: int, state: torch.Tensor,
+                   cache_len: Optional[torch.Tensor], pad_left: Optional[torch.Tensor], B: int, S: int, H: int, D: int, Dv: int
+                   ) -> torch.Tensor:
+    """Linear attention with one fixed decay per head (fp32 [H]) over act(q), act(k), act(v); state fp32 [B, H, D, Dv]; returns the raw
+    read-outs fp32 [B·S, H·Dv]."""
+    _need(y, torch.float32, "y")
+    _need(state, torch.float32, "state")
+    _need(head_decay, torch.float32, "head_decay")
+    L = _lib.lib()
+    out = torch.empty((B * S, H * Dv), dtype=torch.float32, device=y.device)
+    ws = None
+    if S > GLA_FUSED_MAX_TOKENS:
+        ws = torch.empty(int(L.jl_gla_scan_ws_floats(B, S, H, D, Dv)), dtype=torch.float32, device=y.device)
+    _lib.check(L.jl_activated_scan(y.data_ptr(), y.stride(0), q_off, k_off, v_off, head_decay.data_ptr(), act, state.data_ptr(),
+                                   out.data_ptr(), _p(cache_len), _p(pad_left), B, S, H, D, Dv, _p(ws), _stream()), "jl_activated_scan")
+    return out
+
+
+def mlstm_scan(y: torch.Tensor, q_off: int, k_off: int, v_off: int, i_off: int, f_off: int, i_bias: torch.Tensor, f_bias: torch.Tensor,
+               cap: float, q_scale: float, state: torch.Tensor, m_state: torch.Tensor, cache_len: Optional[torch.Tensor],
+               pad_left: Optional[torch.Tensor], B: int, S: int, H: int, D: int, Dv: int) -> "tuple[torch.Tensor, torch.Tensor]":
+    """Matrix memory with exponential gates: advances state fp32 [B, H, D, Dv + 1] (last column: the normaliser n) and the running
+    maximum m_state fp32 [B, H]; returns the raw read-outs fp32 [B·S, H·(Dv + 1)] and the gate numbers fp32 [B·S, 3H]
+    (decay | input scale | exp(−m))."""
+    _need(y, torch.float32, "y")
+    _need(state, torch.float32, "state")
+    _need(m_state, torch.float32, "m_state")
+    L = _lib.lib()
+    M = B * S
+    aux = torch.empty((M, 3 * H), dtype=torch.float32, device=y.device)
+    _lib.check(L.jl_mlstm_gates(y.data_ptr(), y.stride(0), int(i_off), int(f_off), i_bias.data_ptr(), f_bias.data_ptr(), float(cap),
+                                m_state.data_ptr(), aux.data_ptr(), _p(cache_len), _p(pad_left), B, S, H, dtype_code(i_bias.dtype),
+                                _stream()), "jl_mlstm_gates")
+    out = torch.empty((M, H * (Dv + 1)), dtype=torch.float32, device=y.device)
+    ws = None
+    if S > GLA_FUSED_MAX_TOKENS:
+        ws = torch.empty(int(L.jl_gla_scan_ws_floats(B, S, H, D, Dv + 1)), dtype=torch.float32, device=y.device)
+    _lib.check(L.jl_mlstm_scan(y.data_ptr(), y.stride(0), q_off, k_off, v_off, aux.data_ptr(), 3 * H, float(q_scale), state.data_ptr(),
+                               out.data_ptr(), _p(cache_len), _p(pad_left), B, S, H, D, Dv, _p(ws), _stream()), "jl_mlstm_scan")
+    return out, aux
+
+
+def mlstm_finish(o: torch.Tensor, aux: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, H: int, Dv: int, eps: float,
+                 gate_act: int = ACT_SIGMOID) -> torch.Tensor:
+    """Read-outs of `mlstm_scan` → divided by max(|n · q|, exp(−m)) + 1e-6, per-head RMS norm, · w [H·Dv] · act(gate), in w's dtype."""
+    _need(o, torch.float32, "o")
+    _need(gate, torch.float32, "gate")
+    M = o.shape[0]
+    out = torch.empty((M, H * Dv), dtype=w.dtype, device=o.device)
+    _lib.check(_lib.lib().jl_mlstm_finish(o.data_ptr(), aux.data_ptr(), w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), M, H,
+                                          Dv, float(eps), gate_act, dtype_code(w.dtype), _stream()), "jl_mlstm_finish")
+    return out
