@@ -122,4 +122,20 @@ __device__ __forceinline__ void wait_flag(const int* flag, int epoch, int rank, 
 
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
 
+// Four capped scores at once, in place: s -> cap tanh(s / cap) = cap - 2 cap / (1 + e^(2 s / cap)), all in base 2: rate = 2 scale
+// log2(e) / cap turns a raw product into the exponent, cap_log2 = cap log2(e).  The four reciprocals come from one of their
+// denominators' product (special-function throughput bounds the attention kernels); beyond 2^30 the quotient is below the last bit of the
+// result.  Absolute error a few 1e-7 of the cap.
+__device__ __forceinline__ void cap_scores4(float& a, float& b, float& c, float& d, float rate, float cap_log2) {
+  const float ea = 1.0f + exp2f(fminf(a * rate, 30.0f)), eb = 1.0f + exp2f(fminf(b * rate, 30.0f));
+  const float ec = 1.0f + exp2f(fminf(c * rate, 30.0f)), ed = 1.0f + exp2f(fminf(d * rate, 30.0f));
+  const float ab = ea * eb, cd = ec * ed;
+  const float r = __fdividef(-2.0f * cap_log2, ab * cd);
+  const float rab = r * cd, rcd = r * ab;                 // -2 cap / (ea eb), -2 cap / (ec ed)
+  a = fmaf(rab, eb, cap_log2);
+  b = fmaf(rab, ea, cap_log2);
+  c = fmaf(rcd, ed, cap_log2);
+  d = fmaf(rcd, ec, cap_log2);
+}
+
 }  // namespace jl

@@ -146,11 +146,7 @@ __global__ void __launch_bounds__(PM_WARPS * 32) prefill_attn_mma_kernel(const P
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
       const int key = base + 8 * j + 2 * t;
-      if (MASKED && p.cap_log2 > 0.f) {
-        const float twice = 2.0f * p.cap_log2;
-#pragma unroll
-        for (int i = 0; i < 4; ++i) c[j][i] = p.cap_log2 - __fdividef(twice, 1.0f + exp2f(c[j][i] * p.cap_rate));
-      }
+      if (MASKED && p.cap_log2 > 0.f) cap_scores4(c[j][0], c[j][1], c[j][2], c[j][3], p.cap_rate, p.cap_log2);
       c[j][0] = key <= lim0 && (!MASKED || key >= lo0) ? c[j][0] * to_log2 : -INFINITY;
       c[j][1] = key + 1 <= lim0 && (!MASKED || key + 1 >= lo0) ? c[j][1] * to_log2 : -INFINITY;
       c[j][2] = key <= lim1 && (!MASKED || key >= lo1) ? c[j][2] * to_log2 : -INFINITY;

@@ -4,7 +4,8 @@ random weights, plus the time of each kernel of the new design beside the like k
 * ``bench.py --compare folirax`` — Folirax beside LLaMA (`run`),
 * ``bench.py --compare nikonex`` — Nikonex beside Folirax (`run_nikonex`),
 * ``bench.py --compare bazulorn`` — Bazulorn beside Nikonex (`run_bazulorn`),
-* ``bench.py --compare datozen`` — Datozen beside Bazulorn (`run_datozen`).
+* ``bench.py --compare datozen`` — Datozen beside Bazulorn (`run_datozen`),
+* ``bench.py --compare ketolix`` — Ketolix beside Folirax (`run_ketolix`).
 
 Everything is timed with CUDA events on the launching stream after warm-up; per-kernel timings flush L2 (a 256 MB write)
 between iterations, whole-model timings stream more weight bytes than L2 holds.  Fractions are of the measured peaks in
@@ -51,6 +52,17 @@ def llama_config(s: Dict[str, int]) -> Any:
     return LLaMAConfig(vocab_size=s["vocab"], hidden_size=s["width"], intermediate_size=s["ff"],
                        num_hidden_layers=s["layers"], num_attention_heads=s["heads"], num_key_value_heads=s["kv_heads"],
                        max_sequence_length=4096, rms_norm_eps=1e-5)
+
+
+def measured_peaks() -> Dict[str, Any]:
+    """The roofline denominators: HBM copy bandwidth and cuBLAS bf16 burst measured on this kind of GPU, else an earlier measurement."""
+    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+    try:
+        with open(os.path.join(root, "MEASURED_PEAKS.json")) as f:
+            m = json.load(f)
+        return {"hbm_gbs": float(m["hbm_gbs"]), "bf16_tflops": float(m["bf16_tflops"]), "source": "measured"}
+    except (OSError, KeyError, ValueError):
+        return {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
 
 
 class Timer:
@@ -246,14 +258,7 @@ def run(sizes: List[str], prompt_len: int = 2048, steps: int = 64, warmup: int =
     from ..models.hybrid_engine import HybridEngine
 
     dev = torch.device("cuda", torch.cuda.current_device())
-    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
-    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
-    try:
-        with open(os.path.join(root, "MEASURED_PEAKS.json")) as f:
-            m = json.load(f)
-        peaks = {"hbm_gbs": float(m["hbm_gbs"]), "bf16_tflops": float(m["bf16_tflops"]), "source": "measured"}
-    except (OSError, KeyError, ValueError):
-        pass
+    peaks = measured_peaks()
     result: Dict[str, Any] = {"metric": "folirax_vs_llama_equal_size", "data": "synthetic", "dtype": "bf16", "peaks": peaks,
                               "prompt_len": prompt_len, "steps": steps, "warmup": warmup, "sizes": {}}
     for name in sizes:
@@ -493,14 +498,7 @@ def run_nikonex(sizes: List[str], prompt_len: int = 2048, steps: int = 64, warmu
     from ..models.hybrid_engine import HybridEngine
 
     dev = torch.device("cuda", torch.cuda.current_device())
-    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
-    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
-    try:
-        with open(os.path.join(root, "MEASURED_PEAKS.json")) as f:
-            m = json.load(f)
-        peaks = {"hbm_gbs": float(m["hbm_gbs"]), "bf16_tflops": float(m["bf16_tflops"]), "source": "measured"}
-    except (OSError, KeyError, ValueError):
-        pass
+    peaks = measured_peaks()
     result: Dict[str, Any] = {"metric": "nikonex_vs_folirax_equal_size", "data": "synthetic", "dtype": "bf16", "peaks": peaks,
                               "prompt_len": prompt_len, "steps": steps, "warmup": warmup, "sizes": {}}
     for name in sizes:
@@ -753,14 +751,7 @@ def run_bazulorn(sizes: List[str], prompt_len: int = 2048, steps: int = 64, warm
     from ..models.hybrid_engine import HybridEngine
 
     dev = torch.device("cuda", torch.cuda.current_device())
-    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
-    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
-    try:
-        with open(os.path.join(root, "MEASURED_PEAKS.json")) as f:
-            m = json.load(f)
-        peaks = {"hbm_gbs": float(m["hbm_gbs"]), "bf16_tflops": float(m["bf16_tflops"]), "source": "measured"}
-    except (OSError, KeyError, ValueError):
-        pass
+    peaks = measured_peaks()
     result: Dict[str, Any] = {"metric": "bazulorn_vs_nikonex_equal_size", "data": "synthetic", "dtype": "bf16", "peaks": peaks,
                               "prompt_len": prompt_len, "steps": steps, "warmup": warmup, "sizes": {}}
     for name in sizes:
@@ -912,7 +903,7 @@ def _datozen_kernel_table(s: Dict[str, int], dev: torch.device, peaks: Dict[str,
         if masked:
             L.check(L.lib().jl_flash_prefill_masked(qf.data_ptr(), kc.data_ptr(), vc.data_ptr(), pad.data_ptr(), fo.data_ptr(), 1, P, H, G,
                                                     D, T, 0, D ** -0.5, chunk, 1, sink.data_ptr(), gate.data_ptr(), gate.stride(0),
-                                                    vcos.data_ptr(), vsin.data_ptr(), vcos.shape[0], K._stream()), "flash masked")
+                                                    vcos.data_ptr(), vsin.data_ptr(), vcos.shape[0], 0, 0.0, K._stream()), "flash masked")
         else:
             L.check(L.lib().jl_flash_prefill(qf.data_ptr(), kc.data_ptr(), vc.data_ptr(), zero.data_ptr(), pad.data_ptr(), fo.data_ptr(),
                                              1, P, H, G, D, T, 0, D ** -0.5, K._stream()), "flash")
@@ -1001,14 +992,7 @@ def run_datozen(sizes: List[str], prompt_len: int = 2048, steps: int = 64, warmu
     from ..models.hybrid_engine import HybridEngine
 
     dev = torch.device("cuda", torch.cuda.current_device())
-    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
-    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
-    try:
-        with open(os.path.join(root, "MEASURED_PEAKS.json")) as f:
-            m = json.load(f)
-        peaks = {"hbm_gbs": float(m["hbm_gbs"]), "bf16_tflops": float(m["bf16_tflops"]), "source": "measured"}
-    except (OSError, KeyError, ValueError):
-        pass
+    peaks = measured_peaks()
     result: Dict[str, Any] = {"metric": "datozen_vs_bazulorn_equal_size", "data": "synthetic", "dtype": "bf16", "peaks": peaks,
                               "prompt_len": prompt_len, "steps": steps, "warmup": warmup, "sizes": {}}
     for name in sizes:
@@ -1022,5 +1006,201 @@ def run_datozen(sizes: List[str], prompt_len: int = 2048, steps: int = 64, warmu
             torch.cuda.empty_cache()
         if kernels:
             entry["kernels"] = _datozen_kernel_table(s, dev, peaks, prompt_len)
+        result["sizes"][name] = entry
+    return result
+
+
+# --------------------------------------------------------------------------------------------- Ketolix beside Folirax
+def ketolix_config(s: Dict[str, int]) -> Any:
+    """[mlstm, attention, parallel, mlstm] × n at the head counts of the Folirax shape: matrix memory in place of gated linear
+    attention (same 64 × 128 heads), attention with 128-wide heads and a window of 1024, convolved attention of the same heads beside
+    linear attention (64 × 128 heads) in place of the layer that shares keys; three feed-forward matrices that hold what Folirax's two
+    hold."""
+    from ..config import KetolixConfig
+
+    H, G = s["heads"], s["kv_heads"]
+    rot = {"dims": 64, "base": 10000.0}
+    att = {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0, "v_mix": True,
+           "mask": {"size": 1024}, "rot": dict(rot, scaling={"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048})}
+    par = {"left_scale": 0.7, "right_scale": 0.4,
+           "left": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "conv": 4, "mask": {"size": 1024}, "rot": rot},
+           "right": {"heads": H, "dim": 64, "vdim": 128, "decay": [1.0 - 2.0 ** (-1.0 - 7.0 * h / H) for h in range(H)]}}
+    mem = {"heads": H, "dim": 64, "vdim": 128, "gate_cap": 15.0}
+    mlp = {"kind": "dense", "ff": s["ff"] * 2 // 3 // 8 * 8}
+    block = [("mlstm", mem, None), ("attention", att, mlp), ("parallel", par, mlp), ("mlstm", mem, mlp)]
+    return KetolixConfig.from_dict({"architecture": "Ketolix", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5},
+                                    "layers": [{"type": block[i % 4][0], "mixer": block[i % 4][1], "mlp": block[i % 4][2]}
+                                               for i in range(s["layers"])]})
+
+
+def _ketolix_kernel_table(s: Dict[str, int], dev: torch.device, peaks: Dict[str, float], prompt_len: int) -> List[Dict[str, Any]]:
+    """Each kernel that Ketolix adds or extends, at this size, beside the like kernel of the families that came before: ms, achieved
+    rate, the fraction of the measured roofline, and how much farther from it the new kernel is (`distance_ratio`)."""
+    from ..models.mixers import rotary_table
+    from ..ops import _lib as L
+    from ..ops import kernels as K
+    from ..ops import seq_kernels as SK
+
+    t = Timer(dev)
+    hbm, tf = peaks["hbm_gbs"], peaks["bf16_tflops"]
+    W, H, G = s["width"], s["heads"], s["kv_heads"]
+    P, D, Dv, gd, gv, win, cap = prompt_len, 128, 128, 64, 128, 1024, 30.0
+    T = P + 8
+    bf = dict(dtype=torch.bfloat16, device=dev)
+    rows: List[Dict[str, Any]] = []
+
+    def add(name: str, ms: float, like: str, like_ms: float, nbytes: float = 0.0, flops: float = 0.0, like_nbytes: float = 0.0,
+            like_flops: float = 0.0, note: str = "") -> None:
+        work, like_work, unit, peak = (flops, like_flops or flops, "tflops", tf * 1e9) if flops else (nbytes, like_nbytes or nbytes, "gbs",
+                                                                                                     hbm * 1e6)
+        frac, like_frac = work / ms / peak, like_work / like_ms / peak
+        r = {"kernel": name, "ms": round(ms, 4), "like": like, "like_ms": round(like_ms, 4), unit: round(work / ms / (1e9 if flops else 1e6), 2),
+             "frac_bf16_of_measured" if flops else "frac_hbm_of_measured": round(frac, 5), "like_frac": round(like_frac, 5),
+             "distance_ratio": round(like_frac / frac, 2)}
+        if note:
+            r["note"] = note
+        rows.append(r)
+
+    zero = torch.zeros(1, dtype=torch.int32, device=dev)
+    pad = torch.zeros(1, dtype=torch.int32, device=dev)
+    pad8 = torch.zeros(8, dtype=torch.int32, device=dev)
+    last = torch.full((1,), P - 1, dtype=torch.int32, device=dev)
+
+    # ---- residual step
+    x, y1, y2 = torch.randn(P, W, device=dev), torch.randn(P, W, device=dev), torch.randn(P, W, device=dev)
+    w1 = torch.ones(W, **bf)
+    for n, label in ((P, "prompt"), (8, "8 rows")):
+        a, b, c = x[:n].contiguous(), y1[:n].contiguous(), y2[:n].contiguous()
+        like = t.kernel(lambda: SK.postnorm_add(b, w1, a, 1e-5, 0.0, w_next=w1))
+        add(f"postnorm_cast (norm, add, operand copy; {label})", t.kernel(lambda: SK.postnorm_cast(b, w1, a, 1e-5)),
+            "postnorm_add (norm, add, next norm)", like, nbytes=n * W * 14.0)
+        add(f"postnorm_cast of two weighted parts and a bias ({label})",
+            t.kernel(lambda: SK.postnorm_cast(b, w1, a, 1e-5, bias=w1, c1=0.7, y2=c, c2=0.4)), "postnorm_add (norm, add, next norm)", like,
+            nbytes=n * W * 18.0, like_nbytes=n * W * 14.0)
+
+    # ---- attention: convolution, preparation
+    n_qkv = (H + 2 * G) * D
+    yq = torch.randn(P, n_qkv + 8, device=dev) * 0.3
+    qo = torch.empty(P, H * D, **bf)
+    kc, vc = torch.zeros(1, G, T, D, **bf), torch.zeros(1, G, T, Dv, **bf)
+    cos, sin = rotary_table(64, 10000.0, T, dev)
+    qw, kw, lam = torch.ones(H * D, **bf), torch.ones(G * D, **bf), torch.full((), 0.4, **bf)
+    vfirst = yq[:, (H + G) * D:n_qkv]
+    C = (H + G) * D
+    cw, cb = torch.randn(C, 4, **bf), torch.randn(C, device=dev)
+    cst = torch.zeros(8, 3, C, device=dev)
+    for n, B, label in ((P, 1, "prompt"), (8, 8, "8 rows")):
+        S, ln, pd = n // B, zero if B == 1 else last, pad if B == 1 else pad8
+        yy, q_ = yq[:n].contiguous(), qo[:n].contiguous()
+        k_, v_ = (kc, vc) if B == 1 else (torch.zeros(8, G, T, D, **bf), torch.zeros(8, G, T, Dv, **bf))
+        vf = yy[:, (H + G) * D:n_qkv]
+        add(f"causal_conv with a projection bias ({label})",
+            t.kernel(lambda: SK.causal_conv(yy, 0, cw, None, cst, ln, pd, B, S, act=SK.ACT_NONE, in_bias=cb)),
+            "causal_conv + silu (Bazulorn)", t.kernel(lambda: SK.causal_conv(yy, 0, cw, None, cst, ln, pd, B, S)), nbytes=n * C * 8.0)
+        add(f"attn_prep_all (norms over all heads, rotation, mixed values, append; {label})",
+            t.kernel(lambda: SK.attn_prep_all(yy, 0, H * D, C, q_, k_, v_, cos, sin, 64, 0, qw, kw, 1e-5, ln, pd, B, S, H, G, D, Dv,
+                                              v_first=vf, v_lambda=lam)),
+            "attn_prep (rotation, unit-RMS q / k, append; Folirax)",
+            t.kernel(lambda: SK.attn_prep(yy, 0, H * D, C, q_, k_, v_, cos, sin, 64, True, 1e-5, ln, pd, B, S, H, G, D, Dv)),
+            nbytes=n * (n_qkv * 6.0 + G * Dv * 4.0), like_nbytes=n * n_qkv * 6.0)
+
+    # ---- attention proper
+    kc.normal_()
+    vc.normal_()
+    qf = torch.randn(P, H * D, **bf) * 0.3
+    gate = torch.randn(P, H, device=dev)
+    sink = torch.ones(H, device=dev)
+    win_keys, all_keys = float(sum(min(i + 1, win) for i in range(P))), P * (P + 1) / 2.0
+
+    def flash(hd: int, masked: bool, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, softcap: float = 0.0, sinks: bool = False,
+              gated: bool = False) -> torch.Tensor:
+        out = torch.empty_like(q)
+        if masked:
+            L.check(L.lib().jl_flash_prefill_masked(q.data_ptr(), k.data_ptr(), v.data_ptr(), pad.data_ptr(), out.data_ptr(), 1, P, H, G, hd, T,
+                                                    0, hd ** -0.5, 0, int(sinks), sink.data_ptr() if sinks else None,
+                                                    gate.data_ptr() if gated else None, H, None, None, 0, win, softcap, K._stream()), "flash")
+        else:
+            L.check(L.lib().jl_flash_prefill(q.data_ptr(), k.data_ptr(), v.data_ptr(), zero.data_ptr(), pad.data_ptr(), out.data_ptr(), 1, P, H,
+                                             G, hd, T, 0, hd ** -0.5, K._stream()), "flash")
+        return out
+
+    for hd in (128, 64):
+        q_, k_, v_ = qf[:, :H * hd].contiguous(), kc[..., :hd].contiguous(), vc[..., :hd].contiguous()
+        like = t.kernel(lambda: flash(hd, False, q_, k_, v_))
+        kind = "tcgen05" if hd == 128 else "warp-level tensor-core"
+        add(f"window, capped scores, learned sink (prompt, {hd}-wide heads, {kind} kernel)",
+            t.kernel(lambda: flash(hd, True, q_, k_, v_, softcap=cap, sinks=True)), "the same kernel, plain causal attention (LLaMA / Folirax path)",
+            like, flops=4.0 * H * win_keys * hd, like_flops=4.0 * H * all_keys * hd,
+            note="three special-function operations per score against one")
+        add(f"window, gate (prompt, {hd}-wide heads, {kind} kernel)", t.kernel(lambda: flash(hd, True, q_, k_, v_, gated=True)),
+            "the same kernel, plain causal attention (LLaMA / Folirax path)", like, flops=4.0 * H * win_keys * hd,
+            like_flops=4.0 * H * all_keys * hd)
+    add("window, capped scores, sink (prompt, any head size and true float32: attn_rows)",
+        t.kernel(lambda: SK.attn_masked(qf, kc, vc, zero, pad, 1, P, H, G, D, Dv, D ** -0.5, window=win, sink=True, sink_logit=sink, softcap=cap),
+                 reps=3),
+        "attn_rows with a window (Nikonex path)",
+        t.kernel(lambda: SK.attn_windowed(qf, kc, vc, zero, pad, 1, P, H, G, D, Dv, T, D, Dv, win, D ** -0.5), reps=3),
+        flops=4.0 * H * win_keys * D)
+    q1, g1 = qf[:1].contiguous(), gate[:1].contiguous()
+    add("window, capped scores, sink (one token: attn_split + attn_merge)",
+        t.kernel(lambda: SK.attn_masked(q1, kc, vc, last, pad, 1, 1, H, G, D, Dv, D ** -0.5, window=win, sink=True, sink_logit=sink, softcap=cap)),
+        "attn_split + attn_merge with a window (Nikonex path)",
+        t.kernel(lambda: SK.attn_windowed(q1, kc, vc, last, pad, 1, 1, H, G, D, Dv, T, D, Dv, win, D ** -0.5)),
+        nbytes=min(win, P) * G * (D + Dv) * 2.0)
+
+    # ---- scans: activated linear attention and matrix memory beside retention (fixed decays) and the state space scan (decay per token)
+    n_in = 2 * H * gd + 2 * H * gv + 2 * H
+    ys = torch.randn(P, (n_in + 7) // 8 * 8, device=dev) * 0.3
+    q_off, k_off, v_off, g_off = 0, H * gd, 2 * H * gd, 2 * H * gd + H * gv
+    dec = torch.full((H,), 0.95, device=dev)
+    ib, fb, alog, dtb = torch.zeros(H, **bf), torch.full((H,), 3.0, **bf), torch.zeros(H, **bf), torch.zeros(H, **bf)
+    for n, B, label in ((P, 1, "prompt"), (8 * P, 8, "prompt, 8 rows"), (8, 8, "one token, 8 rows")):
+        S, ln, pd = n // B, zero if n > 8 else last, pad if B == 1 else pad8
+        yy = ys[:n].contiguous() if n <= P else ys.repeat(8, 1)
+        st, st1, ms_ = torch.zeros(B, H, gd, gv, device=dev), torch.zeros(B, H, gd, gv + 1, device=dev), torch.zeros(B, H, device=dev)
+        fl, by = 4.0 * n * H * gd * gv, n * H * (gd * 2 + gv * 2) * 4.0 + (2.0 * st.numel() * 4 if S == 1 else 0.0)
+        work: Dict[str, float] = {"nbytes": by} if S == 1 else {"flops": fl}
+        ret = t.kernel(lambda: SK.retention_scan(yy, q_off, k_off, v_off, dec, cos, sin, 64, 0, 0.125, st, ln, pd, B, S, H, gd, gv), reps=5)
+        ssd = t.kernel(lambda: SK.ssd_scan(yy, g_off, dtb, alog, yy, q_off, k_off, v_off, H, st, ln, pd, B, S, H, gd, gv), reps=5)
+        add(f"activated scan (silu q, k, v; fixed decays; {label})",
+            t.kernel(lambda: SK.activated_scan(yy, q_off, k_off, v_off, dec, SK.ACT_SILU, st, ln, pd, B, S, H, gd, gv), reps=5),
+            "retention scan (Nikonex)", ret, **work)
+        add(f"matrix memory (gates, scan with the normaliser column; {label})",
+            t.kernel(lambda: SK.mlstm_scan(yy, q_off, k_off, v_off, g_off + H * gv, g_off + H * gv + H, ib, fb, 15.0, 0.125, st1, ms_, ln, pd, B, S,
+                                           H, gd, gv), reps=5), "state space scan (gates, scan; Bazulorn)", ssd, **work)
+
+    # ---- gated read-outs
+    for n, label in ((P, "prompt"), (8, "8 rows")):
+        o, o1, gt = torch.randn(n, H * gv, device=dev), torch.randn(n, H * (gv + 1), device=dev), torch.randn(n, H * gv, device=dev)
+        aux, wv, wf = torch.rand(n, 3 * H, device=dev), torch.ones(gv, **bf), torch.ones(H * gv, **bf)
+        like = t.kernel(lambda: SK.headnorm_gate(o, wv, gt, H, gv, 1e-5, SK.ACT_SILU))
+        add(f"rownorm_gate (norm over all heads, weight, sigmoid gate; {label})", t.kernel(lambda: SK.rownorm_gate(o, wf, gt, 1e-5)),
+            "headnorm_gate (norm per head, silu gate; Folirax)", like, nbytes=n * H * gv * 10.0)
+        add(f"mlstm_finish (division, norm per head, weight, sigmoid gate; {label})",
+            t.kernel(lambda: SK.mlstm_finish(o1, aux, wf, gt, H, gv, 1e-5)), "headnorm_gate (norm per head, silu gate; Folirax)", like,
+            nbytes=n * H * gv * 10.0)
+    return rows
+
+
+def run_ketolix(sizes: List[str], prompt_len: int = 2048, steps: int = 64, warmup: int = 8, batches: List[int] = (1, 8),
+                kernels: bool = True) -> Dict[str, Any]:
+    """Ketolix beside the closest existing design, Folirax (sequential sublayers, dense feed-forward, softmax attention among linear
+    recurrences), at equal width, depth, head counts and feed-forward parameters."""
+    from ..models.hybrid_engine import HybridEngine
+
+    dev = torch.device("cuda", torch.cuda.current_device())
+    peaks = measured_peaks()
+    result: Dict[str, Any] = {"metric": "ketolix_vs_folirax_equal_size", "data": "synthetic", "dtype": "bf16", "peaks": peaks,
+                              "prompt_len": prompt_len, "steps": steps, "warmup": warmup, "sizes": {}}
+    for name in sizes:
+        s = SIZES[name]
+        entry: Dict[str, Any] = {"shape": s}
+        for label, cfg in (("ketolix", ketolix_config(s)), ("folirax", folirax_config(s))):
+            eng = HybridEngine.random_init(cfg, dev, seed=0)
+            entry[label] = _model_times(eng, s["vocab"], prompt_len, list(batches), steps, warmup)
+            del eng
+            torch.cuda.empty_cache()
+        if kernels:
+            entry["kernels"] = _ketolix_kernel_table(s, dev, peaks, prompt_len)
         result["sizes"][name] = entry
     return result
