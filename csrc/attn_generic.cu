@@ -4,12 +4,13 @@
 //  * attn_prep_kernel   — interleaved-pair rotary embedding on the first `rot` channels of each head (pair 2i, 2i+1;
 //    the rest pass through), then optional weight-free unit-RMS scaling of q and k per head, append of k / v to the
 //    cache [B][G][T][D] / [B][G][T][Dv].  Token (b, s) goes to slot *cache_len + s at position slot - pad_left[b].
-//    A layer that reads another layer's keys and values runs it for the queries only.
+//    A layer that reads another layer's keys and values runs it for the queries only.  Queries can grow with their position
+//    (a factor 1 + coef ln(1 + floor((position + 1) / every)) on the finished query).
 //  * attn_prep_all_kernel — the same for designs that norm q (and k) over all heads together and mix the values with another
 //    layer's; two CTAs per token.
 //  * attn_rows_kernel   — 16 queries of one head per CTA against key / value tiles of 32 rows staged in shared memory
 //    (one key per lane for the scores, one value column per lane for the output), online softmax in fp32, causal over
-//    slots [pad_left[b], slot], optional per-head output gate sigmoid(g).  Prompts of any length; exact path for
+//    slots [pad_left[b], slot], optional output gate sigmoid(g) per head or per channel.  Prompts of any length; exact path for
 //    float32 and for head sizes the tensor-core kernels are not built for.
 //  * attn_decode_kernel — one CTA per (row, head) for a single new token: its warps take interleaved blocks of 32 keys
 //    and merge their (max, sum, output) triples in shared memory (what runs when the caller brings no scratch).
@@ -45,7 +46,12 @@ struct PrepParams {
                                     // rotation, shared by the heads; nullptr: none
   const float* vcos; const float* vsin; int v_max_pos, v_layout;   // [v_max_pos][Dv/2]: values are rotated at their own position over all
                                     // Dv channels before they are cached (pairs as v_layout says); nullptr: cached as they are
+  float q_coef; int q_every;        // q_every > 0: the finished query is multiplied by 1 + q_coef ln(1 + floor((position + 1) / q_every))
 };
+
+__device__ __forceinline__ float query_factor(const PrepParams& p, int pos) {
+  return p.q_every > 0 && pos >= 0 ? 1.0f + p.q_coef * logf((float)((pos + 1) / p.q_every + 1)) : 1.0f;
+}
 
 constexpr int AP_WARPS = 4;      // heads per CTA of the preparation kernel (one warp each)
 
@@ -90,6 +96,7 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prep_kernel(PrepParams p, 
     return;
   }
   const bool is_q = head < p.H;
+  const float grow = is_q ? query_factor(p, slot - (p.pad_left ? p.pad_left[b] : 0)) : 1.0f;
   const int col = is_q ? p.q_off + head * p.D : p.k_off + (head - p.H) * p.D;
   const float* src = yr + col;
   const float* bs = p.bias ? p.bias + col : nullptr;
@@ -106,7 +113,7 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prep_kernel(PrepParams p, 
       for (int c = lane; c < p.D; c += 32) { const float v = src[c] + (bs ? bs[c] : 0.0f); ss += v * v; }
       r = 1.0f / sqrtf(warp_sum(ss) / (float)p.D + p.eps);
     }
-    auto val = [&](int c) { const float v = src[c] + (bs ? bs[c] : 0.0f); return w ? v * r * to_f(w[c]) : v; };
+    auto val = [&](int c) { const float v = src[c] + (bs ? bs[c] : 0.0f); return (w ? v * r * to_f(w[c]) : v) * grow; };
     const int half = p.rot / 2;
     for (int i = lane; i < half; i += 32) {
       const int c0 = p.layout ? i : 2 * i, c1 = p.layout ? i + half : 2 * i + 1;
@@ -119,7 +126,7 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prep_kernel(PrepParams p, 
   }
   const int npairs = p.D / 2 + (p.D & 1);
   // pass 1 rotates and sums the squares, pass 2 rotates again (L1 hits) and writes the scaled values
-  float r = 1.0f;
+  float r = grow;
   for (int pass = p.unit_norm ? 0 : 1; pass < 2; ++pass) {
     float ss = 0.0f;
     for (int i = lane; i < npairs; i += 32) {
@@ -136,13 +143,14 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prep_kernel(PrepParams p, 
         if (c1 < p.D) dst[c1] = from_f<T>(v * r);
       }
     }
-    if (pass == 0) r = 1.0f / sqrtf(warp_sum(ss) / (float)p.D + p.eps);
+    if (pass == 0) r = grow / sqrtf(warp_sum(ss) / (float)p.D + p.eps);
   }
 }
 
 // Latent attention, preparation: the fused down-projection row y holds the query latent (q_rank columns at q_off) and the
 // key/value latent followed by one rotated key part shared by all heads (kv_rank + rot_dim columns at kv_off).  Both latents
-// are RMS-normed with a plain weight; the key part gets the rotary embedding of the token's position on its first `rot`
+// are RMS-normed with a plain weight (a design without a query latent passes no weight: the query columns, all heads' queries, are
+// only brought into the operand type); the key part gets the rotary embedding of the token's position on its first `rot`
 // channels.  The normed query latent goes to cq [M][q_rank]; the normed key/value latent and the rotated key part are
 // appended as ONE cache row [kv_rank | rot_dim] at slot *cache_len + s — all that this kind of layer keeps per token.
 struct LatentPrepParams {
@@ -153,6 +161,7 @@ struct LatentPrepParams {
   int B, S, T;
   const int* cache_len; const int* pad_left;
   void* c_out; void* kr_out;        // optional token-major copies of what was appended: latent [M][kv_rank], key part [M][rot_dim]
+  int q_vec;                        // queries without a norm: 16-byte reads of their columns are aligned
 };
 
 template <typename T>
@@ -166,7 +175,15 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepParams p, co
   int pos = slot - (p.pad_left ? p.pad_left[b] : 0);
   pos = pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos);
   const float* yr = p.y + (size_t)m * p.ldy;
-  if (p.q_rank > 0) {
+  if (p.q_rank > 0 && wq == nullptr) {
+    T* dst = cq + (size_t)m * p.q_rank;
+    const float* src = yr + p.q_off;
+    if (p.q_vec) {
+      for (int i = 4 * threadIdx.x; i < p.q_rank; i += 4 * blockDim.x) { float v[4]; load4(src + i, v); store4(dst + i, v); }
+    } else {
+      for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) dst[i] = from_f<T>(src[i]);
+    }
+  } else if (p.q_rank > 0) {
     float ss = 0.0f;
     for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) { const float v = yr[p.q_off + i]; ss += v * v; }
     const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)p.q_rank + p.eps);
@@ -334,7 +351,7 @@ struct AttnParams {
   float scale;
   const int* cache_len;             // slots already filled BEFORE this call's tokens (device scalar); nullptr = 0
   const int* pad_left;
-  const float* gate; int ldg;       // fp32 pre-activation of the per-head output gate (column h of row m), or nullptr
+  const float* gate; int ldg;       // fp32 pre-activation of the output gate of row m: column h (one per head), with gate_cols column h * Dv + c; or nullptr
   int sink;                         // 1: the softmax denominator has one more term exp(0) (a key with score 0 and no value)
   float* out32;                     // fp32 output [M][H][Dv] instead of `out` (what a later fp32 step reads), or nullptr
   int chunk;                        // > 0: positions (slot - pad_left) form blocks of `chunk`; a query sees the keys of its own block only
@@ -342,7 +359,13 @@ struct AttnParams {
   const float* vcos; const float* vsin; int v_max_pos, v_layout;   // [v_max_pos][Dv/2]: the cached values were rotated at their own
                                     // positions; every head's sum is rotated back by the query's position (pairs as v_layout)
   float softcap;                    // > 0: scores become softcap * tanh(score / softcap)
+  int gate_cols;                    // 1: the output gate has one number per channel instead of one per head
 };
+
+// factor of the output gate on value column c of head h of row m (the whole row's factor when the gate is per head: any c)
+__device__ __forceinline__ float attn_gate(const AttnParams& p, size_t m, int h, int c) {
+  return sigmoid_f(p.gate[m * p.ldg + (p.gate_cols ? h * p.Dv + c : h)]);
+}
 
 __device__ __forceinline__ float attn_score(float dot, float scale, float softcap) {
   const float s = dot * scale;
@@ -586,11 +609,11 @@ __global__ void __launch_bounds__(AR_WARPS * 32) attn_rows_kernel(AttnParams p, 
       __syncwarp();
       continue;
     }
-    if (p.gate) gmul *= sigmoid_f(p.gate[(size_t)m * p.ldg + h]);
+    if (p.gate && !p.gate_cols) gmul *= attn_gate(p, m, h, 0);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = lane + 32 * i;
-      if (c < p.Dv) attn_store<T>(p, out, ((size_t)m * p.H + h) * p.Dv + c, acc[qi][i] * gmul);
+      if (c < p.Dv) attn_store<T>(p, out, ((size_t)m * p.H + h) * p.Dv + c, acc[qi][i] * (p.gate_cols ? gmul * attn_gate(p, m, h, c) : gmul));
     }
   }
 }
@@ -645,11 +668,11 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_kernel(AttnParams p
     attn_finish_row<T>(p, out, ((size_t)b * p.H + h) * p.Dv, part, hi - lo_seq, gate, threadIdx.x, blockDim.x);
     return;
   }
-  if (p.gate) gmul *= sigmoid_f(p.gate[(size_t)b * p.ldg + h]);
+  if (p.gate && !p.gate_cols) gmul *= attn_gate(p, b, h, 0);
   for (int c = threadIdx.x; c < p.Dv; c += blockDim.x) {
     float o = 0.0f;
     for (int w = 0; w < AD_WARPS; ++w) if (ml[2 * w] != -INFINITY) o += part[w * p.Dv + c] * expf(ml[2 * w] - mall);
-    attn_store<T>(p, out, ((size_t)b * p.H + h) * p.Dv + c, o * gmul);
+    attn_store<T>(p, out, ((size_t)b * p.H + h) * p.Dv + c, o * (p.gate_cols ? gmul * attn_gate(p, b, h, c) : gmul));
   }
 }
 
@@ -802,12 +825,12 @@ __global__ void attn_merge_kernel(AttnParams p, const float* __restrict__ part, 
     attn_finish_row<T>(p, out, ((size_t)b * p.H + h) * p.Dv, orow, hi - (p.pad_left ? p.pad_left[b] : 0), gate, threadIdx.x, blockDim.x);
     return;
   }
-  if (p.gate) gmul *= sigmoid_f(p.gate[(size_t)b * p.ldg + h]);
+  if (p.gate && !p.gate_cols) gmul *= attn_gate(p, b, h, 0);
   for (int c = threadIdx.x; c < p.Dv; c += blockDim.x) {
     float o = 0.0f;
 #pragma unroll 8
     for (int zz = 0; zz < splits; ++zz) o = fmaf(src[(size_t)zz * (p.Dv + 2) + 2 + c], wz[zz], o);
-    attn_store<T>(p, out, ((size_t)b * p.H + h) * p.Dv + c, o * gmul);
+    attn_store<T>(p, out, ((size_t)b * p.H + h) * p.Dv + c, o * (p.gate_cols ? gmul * attn_gate(p, b, h, c) : gmul));
   }
 }
 
@@ -832,6 +855,7 @@ static int attn_prep_launch(PrepParams p, void* q_out, void* k_cache, void* v_ca
   JL_CHECK_ARG(p.rot >= 0 && p.rot <= p.D && p.rot % 2 == 0, "jl_attn_prep: rot=%d must be even and <= D=%d", p.rot, p.D);
   JL_CHECK_ARG(p.k_off >= 0 || (k_cache == nullptr && v_cache == nullptr), "jl_attn_prep: queries-only call takes no caches");
   JL_CHECK_ARG(p.layout == 0 || p.layout == 1, "jl_attn_prep: layout %d", p.layout);
+  JL_CHECK_ARG(p.q_every >= 0, "jl_attn_prep: query growth every %d positions", p.q_every);
   JL_CHECK_ARG((p.qw == nullptr) == (p.kw == nullptr), "jl_attn_prep: the q and k norm weights come together");
   JL_CHECK_ARG(!(p.unit_norm && (p.qw != nullptr || p.layout != 0)),
                "jl_attn_prep: unit-RMS scaling after the rotation goes with interleaved pairs and no weighted norm");
@@ -851,20 +875,21 @@ extern "C" JL_API int jl_attn_prep(const float* y, int ldy, int q_off, int k_off
                                    float eps, const int* cache_len, const int* pad_left, int B, int S, int H, int G, int D, int Dv,
                                    int T_cap, const float* bias, int v_norm, int v_token_major, int dtype, void* stream) {
   PrepParams p{y, ldy, q_off, k_off, v_off, B, S, H, G, D, Dv, T_cap, rot, cos_t, sin_t, max_pos, unit_norm, eps, cache_len, pad_left,
-               bias, v_norm, v_token_major, 0, nullptr, nullptr, nullptr, nullptr, 0, 0};
+               bias, v_norm, v_token_major, 0, nullptr, nullptr, nullptr, nullptr, 0, 0, 0.0f, 0};
   return attn_prep_launch(p, q_out, k_cache, v_cache, dtype, stream);
 }
 
 // The same with the newer pieces: `layout` of the rotated q / k pairs, an RMS norm with weights q_norm_w / k_norm_w [D] before the
-// rotation, and values rotated at their own position with the tables v_cos / v_sin [v_max_pos][Dv/2] (pairs as v_layout).
+// rotation, values rotated at their own position with the tables v_cos / v_sin [v_max_pos][Dv/2] (pairs as v_layout), and (q_every > 0)
+// queries multiplied by 1 + q_coef ln(1 + floor((position + 1) / q_every)).
 extern "C" JL_API int jl_attn_prep_ex(const float* y, int ldy, int q_off, int k_off, int v_off, void* q_out, void* k_cache,
                                       void* v_cache, const float* cos_t, const float* sin_t, int max_pos, int rot, int layout,
                                       int unit_norm, const void* q_norm_w, const void* k_norm_w, float eps, const float* v_cos,
                                       const float* v_sin, int v_max_pos, int v_layout, const int* cache_len, const int* pad_left,
                                       int B, int S, int H, int G, int D, int Dv, int T_cap, const float* bias, int v_norm,
-                                      int v_token_major, int dtype, void* stream) {
+                                      int v_token_major, float q_coef, int q_every, int dtype, void* stream) {
   PrepParams p{y, ldy, q_off, k_off, v_off, B, S, H, G, D, Dv, T_cap, rot, cos_t, sin_t, max_pos, unit_norm, eps, cache_len, pad_left,
-               bias, v_norm, v_token_major, layout, q_norm_w, k_norm_w, v_cos, v_sin, v_max_pos, v_layout};
+               bias, v_norm, v_token_major, layout, q_norm_w, k_norm_w, v_cos, v_sin, v_max_pos, v_layout, q_coef, q_every};
   return attn_prep_launch(p, q_out, k_cache, v_cache, dtype, stream);
 }
 
@@ -905,18 +930,19 @@ static int attn_launch(const void* q, const void* k_cache, const void* v_cache, 
                        int ldv, int window, float scale, float* scratch, int splits, int dtype, void* stream,
                        long long k_bs = 0, long long k_hs = 0, long long v_bs = 0, long long v_hs = 0, int sink = 0,
                        float* out32 = nullptr, int chunk = 0, const float* sink_logit = nullptr, const float* vcos = nullptr,
-                       const float* vsin = nullptr, int v_max_pos = 0, int v_layout = 0, float softcap = 0.0f) {
+                       const float* vsin = nullptr, int v_max_pos = 0, int v_layout = 0, float softcap = 0.0f, int gate_cols = 0) {
   JL_CHECK_ARG(B >= 1 && S >= 1 && G >= 1 && H % G == 0, "jl_attn_generic: H=%d not a multiple of G=%d", H, G);
   JL_CHECK_ARG(Dv <= 32 * AT_MAXV, "jl_attn_generic: value size %d above %d", Dv, 32 * AT_MAXV);
   JL_CHECK_ARG(ldk >= D && ldv >= Dv && window >= 0, "jl_attn_generic: bad pitch %d / %d or window %d", ldk, ldv, window);
   if (k_bs == 0 && k_hs == 0) { k_hs = (long long)T_cap * ldk; k_bs = k_hs * G; }
   if (v_bs == 0 && v_hs == 0) { v_hs = (long long)T_cap * ldv; v_bs = v_hs * G; }
   JL_CHECK_ARG(softcap >= 0.0f, "jl_attn_generic: softcap %f", softcap);
+  JL_CHECK_ARG(!gate_cols || (gate != nullptr && vcos == nullptr && ldg >= H * Dv), "jl_attn_generic: a gate per channel goes with values as they are");
   JL_CHECK_ARG(chunk >= 0 && (sink_logit == nullptr || sink), "jl_attn_generic: chunk %d, a sink logit without a sink", chunk);
   JL_CHECK_ARG(vcos == nullptr || (vsin != nullptr && Dv % 2 == 0 && v_max_pos >= 1 && (v_layout == 0 || v_layout == 1)),
                "jl_attn_generic: rotated values need both tables and an even Dv=%d", Dv);
   AttnParams p{B, S, H, G, D, Dv, T_cap, ldk, ldv, k_bs, k_hs, v_bs, v_hs, window, scale, cache_len, pad_left, gate, ldg, sink, out32,
-               chunk, sink_logit, vcos, vsin, v_max_pos, v_layout, softcap};
+               chunk, sink_logit, vcos, vsin, v_max_pos, v_layout, softcap, gate_cols};
   cudaStream_t st = (cudaStream_t)stream;
   if (S == 1 && scratch != nullptr && splits >= 1 && splits <= 64) {
     const int dp = ((D + 3) & ~3) + 4;
@@ -974,10 +1000,10 @@ extern "C" JL_API int jl_attn_windowed(const void* q, const void* k_cache, const
                      scratch, splits, dtype, stream, k_bs, k_hs, v_bs, v_hs, sink, out32);
 }
 
-// Everything the attention kernels take: gate (fp32 pre-activation, column h of row m, pitch ldg), window, blocks of `chunk`
+// Everything the attention kernels take: gate (fp32 pre-activation, column h of row m, with gate_cols column h * Dv + c, pitch ldg), window, blocks of `chunk`
 // positions, capped scores (softcap > 0), a sink (score 0, or sink_logit[h]), values cached rotated (v_cos / v_sin [v_max_pos][Dv/2], pairs as v_layout).
 extern "C" JL_API int jl_attn_masked(const void* q, const void* k_cache, const void* v_cache, void* out, const float* gate, int ldg,
-                                     const int* cache_len, const int* pad_left, int B, int S, int H, int G, int D, int Dv, int T_cap,
+                                     int gate_cols, const int* cache_len, const int* pad_left, int B, int S, int H, int G, int D, int Dv, int T_cap,
                                      int ldk, int ldv, long long k_bs, long long k_hs, long long v_bs, long long v_hs, int window,
                                      int chunk, float scale, float softcap, float* scratch, int splits, int sink, const float* sink_logit,
                                      const float* v_cos, const float* v_sin, int v_max_pos, int v_layout, float* out32, int dtype,
@@ -985,7 +1011,7 @@ extern "C" JL_API int jl_attn_masked(const void* q, const void* k_cache, const v
   JL_CHECK_ARG(out != nullptr || out32 != nullptr, "jl_attn_masked: no output");
   return attn_launch(q, k_cache, v_cache, out, gate, ldg, cache_len, pad_left, B, S, H, G, D, Dv, T_cap, ldk, ldv, window, scale,
                      scratch, splits, dtype, stream, k_bs, k_hs, v_bs, v_hs, sink, out32, chunk, sink_logit, v_cos, v_sin, v_max_pos,
-                     v_layout, softcap);
+                     v_layout, softcap, gate_cols);
 }
 
 extern "C" JL_API int jl_latent_prep(const float* y, int ldy, int q_off, int q_rank, int kv_off, int kv_rank, int rot_dim, int rot,
@@ -997,7 +1023,8 @@ extern "C" JL_API int jl_latent_prep(const float* y, int ldy, int q_off, int q_r
   JL_CHECK_ARG(rot >= 0 && rot <= rot_dim && rot % 2 == 0, "jl_latent_prep: rot=%d must be even and <= rot_dim=%d", rot, rot_dim);
   JL_CHECK_ARG(layout == 0 || layout == 1, "jl_latent_prep: layout %d", layout);
   LatentPrepParams p{y, ldy, q_off, q_rank, kv_off, kv_rank, rot_dim, rot, layout, cos_t, sin_t, max_pos, eps, B, S, T_cap,
-                     cache_len, pad_left, c_out, kr_out};
+                     cache_len, pad_left, c_out, kr_out,
+                     q_rank % 4 == 0 && ldy % 4 == 0 && q_off % 4 == 0 && (((uintptr_t)y | (uintptr_t)cq) % 16) == 0};
   JL_DISPATCH_DTYPE(dtype, JL_LAUNCH_PDL(latent_prep_kernel<T>, dim3(B * S), dim3(128), 0, (cudaStream_t)stream, p, (const T*)wq_norm,
                                          (const T*)wkv_norm, (T*)cq, (T*)cache));
   JL_CUDA(cudaGetLastError());

@@ -38,12 +38,14 @@ struct FlashParams {
   int chunk;                        // > 0: positions (slot - pad_left) form blocks of `chunk`; a query sees the keys of its own block only
   int sink;                         // the softmax denominator has one more term exp(sink_logit[h]) (exp(0) without logits)
   const float* sink_logit;          // fp32 [nh] or nullptr
-  const float* gate; int ldg;       // fp32 pre-activation of a sigmoid per (token, head) on the output (column h of row m), or nullptr
+  const float* gate; int ldg;       // fp32 pre-activation of a sigmoid on the output of row m, or nullptr: column h (one per head), with gate_cols
+                                    // column h * 128 + d (16-byte aligned rows)
   const float* vcos; const float* vsin; int v_max_pos;   // [v_max_pos][64]: the cached values were rotated at their own positions over
                                     // all 128 channels (pairs m, m + 64); every row of the output is rotated back by its position
   int window;                       // > 0: a query sees itself and the window - 1 slots before it
   float cap_log2, cap_rate;         // cap_log2 > 0: scores are capped, s -> cap tanh(s / cap): cap log2(e) and the factor 2 scale log2(e) / cap
                                     // that turns a raw product into the exponent of e^(2 s / cap) in base 2
+  int gate_cols;                    // 1: the gate has one number per output channel
 };
 
 __device__ __forceinline__ void cap_bits4(uint32_t* v, float rate, float cap_log2) {
@@ -537,7 +539,9 @@ flash_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
     }
     uint4* dst = reinterpret_cast<uint4*>(p.out + ((size_t)(b * p.S + q0 + r) * p.nh + h) * FA_HD);
     const bool row_on = q0 + r < p.S;
-    if (MASKED && p.gate != nullptr && row_on) inv *= 1.0f / (1.0f + __expf(-p.gate[(size_t)(b * p.S + q0 + r) * p.ldg + h]));
+    const bool gate_row = MASKED && p.gate != nullptr && p.gate_cols;
+    const float* gate_src = gate_row && row_on ? p.gate + (size_t)(b * p.S + q0 + r) * p.ldg + h * FA_HD : nullptr;
+    if (MASKED && p.gate != nullptr && !p.gate_cols && row_on) inv *= 1.0f / (1.0f + __expf(-p.gate[(size_t)(b * p.S + q0 + r) * p.ldg + h]));
     if (MASKED && p.vcos != nullptr) {
       // the row's sum is turned back by its position: channel m pairs with m + 64, so column chunks 0 / 1 meet chunks 2 / 3
       int pos = q_slot - pad;
@@ -596,6 +600,16 @@ flash_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
 #pragma unroll
         for (int i = 0; i < 32; ++i) o[i] = 0u;
       }
+      if (gate_src != nullptr) {                             // 128 bytes of the row's gate per chunk of 32 channels
+        const float4* g4 = reinterpret_cast<const float4*>(gate_src + c * 32);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+          const float4 gv = __ldg(g4 + k);
+          const float gs[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+          for (int e = 0; e < 4; ++e) o[4 * k + e] = __float_as_uint(__fdividef(__uint_as_float(o[4 * k + e]), 1.0f + __expf(-gs[e])));
+        }
+      }
       if (q0 + r < p.S) {
 #pragma unroll
         for (int i = 0; i < 4; ++i)
@@ -642,35 +656,38 @@ extern "C" JL_API int jl_flash_prefill_occupancy(int smem_override) {
 
 static int flash_launch(const void* q, const void* k_cache, const void* v_cache, const int* pad_left, void* out, int B, int S, int nh,
                         int nkv, int hd, int T, int start, float scale, void* stream, int chunk, int sink, const float* sink_logit,
-                        const float* gate, int ldg, const float* vcos, const float* vsin, int v_max_pos, int window, float softcap);
+                        const float* gate, int ldg, int gate_cols, const float* vcos, const float* vsin, int v_max_pos, int window, float softcap);
 
 extern "C" JL_API int jl_flash_prefill(const void* q, const void* k_cache, const void* v_cache,
                                        const int* cache_len_ptr, const int* pad_left, void* out, int B, int S,
                                        int nh, int nkv, int hd, int T, int start, float scale, void* stream) {
   (void)cache_len_ptr;
-  return flash_launch(q, k_cache, v_cache, pad_left, out, B, S, nh, nkv, hd, T, start, scale, stream, 0, 0, nullptr, nullptr, 0, nullptr,
+  return flash_launch(q, k_cache, v_cache, pad_left, out, B, S, nh, nkv, hd, T, start, scale, stream, 0, 0, nullptr, nullptr, 0, 0, nullptr,
                       nullptr, 0, 0, 0.0f);
 }
 
 // The tcgen05 kernel (128-wide heads) with blocks of `chunk` positions, a window, capped scores, a sink in the denominator (logit per head), a sigmoid gate
-// per (token, head) and the turn back of values that were cached rotated at their own positions (pairs m, m + 64).  64-wide heads
+// per (token, head) or (gate_cols) per (token, channel) and the turn back of values that were cached rotated at their own positions (pairs m, m + 64).  64-wide heads
 // run the warp-level tensor-core kernel with the same options (no value rotation).
 extern "C" JL_API int jl_flash_prefill_masked(const void* q, const void* k_cache, const void* v_cache, const int* pad_left, void* out,
                                               int B, int S, int nh, int nkv, int hd, int T, int start, float scale, int chunk,
-                                              int sink, const float* sink_logit, const float* gate, int ldg, const float* v_cos,
-                                              const float* v_sin, int v_max_pos, int window, float softcap, void* stream) {
+                                              int sink, const float* sink_logit, const float* gate, int ldg, int gate_cols,
+                                              const float* v_cos, const float* v_sin, int v_max_pos, int window, float softcap,
+                                              void* stream) {
   JL_CHECK_ARG(hd == FA_HD || (hd == 64 && v_cos == nullptr), "jl_flash_prefill_masked: head_dim=%d (128, and 64 without rotated values)", hd);
   JL_CHECK_ARG(window >= 0 && softcap >= 0.0f, "jl_flash_prefill_masked: window %d, softcap %f", window, softcap);
   JL_CHECK_ARG(chunk >= 0 && (sink_logit == nullptr || sink) && (gate == nullptr || ldg >= nh),
                "jl_flash_prefill_masked: chunk %d, sink %d, gate pitch %d", chunk, sink, ldg);
   JL_CHECK_ARG(v_cos == nullptr || (v_sin != nullptr && v_max_pos >= 1), "jl_flash_prefill_masked: rotated values need both tables");
+  JL_CHECK_ARG(!gate_cols || (gate != nullptr && v_cos == nullptr && ldg >= nh * hd && ldg % 4 == 0 && (uintptr_t)gate % 16 == 0),
+               "jl_flash_prefill_masked: a gate per channel needs 16-byte rows (pitch %d) and values as they are", ldg);
   return flash_launch(q, k_cache, v_cache, pad_left, out, B, S, nh, nkv, hd, T, start, scale, stream, chunk, sink, sink_logit, gate, ldg,
-                      v_cos, v_sin, v_max_pos, window, softcap);
+                      gate_cols, v_cos, v_sin, v_max_pos, window, softcap);
 }
 
 static int flash_launch(const void* q, const void* k_cache, const void* v_cache, const int* pad_left, void* out, int B, int S, int nh,
                         int nkv, int hd, int T, int start, float scale, void* stream, int chunk, int sink, const float* sink_logit,
-                        const float* gate, int ldg, const float* vcos, const float* vsin, int v_max_pos, int window, float softcap) {
+                        const float* gate, int ldg, int gate_cols, const float* vcos, const float* vsin, int v_max_pos, int window, float softcap) {
   const bool extras = chunk > 0 || window > 0 || softcap > 0.0f || sink || gate != nullptr || vcos != nullptr;
   // 64-wide heads (1B-class LLaMA-architecture models) go to the warp-level tensor-core kernel (prefill_attn_mma.cu);
   // JLLAMA_PREFILL_MMA=1 sends head_dim 128 there too (A/B against the tcgen05 kernel below)
@@ -679,7 +696,7 @@ static int flash_launch(const void* q, const void* k_cache, const void* v_cache,
     return jl_prefill_attn_mma(q, k_cache, v_cache, pad_left, out, B, S, nh, nkv, hd, T, start, scale, stream);
   if (hd == 64)
     return jl_prefill_attn_mma_masked(q, k_cache, v_cache, pad_left, out, B, S, nh, nkv, hd, T, start, scale, window, chunk, softcap, sink,
-                                      sink_logit, gate, ldg, stream);
+                                      sink_logit, gate, ldg, gate_cols, stream);
   JL_CHECK_ARG(hd == FA_HD, "jl_flash_prefill: head_dim=%d (64 and 128 are built)", hd);
   JL_CHECK_ARG(nkv > 0 && nh % nkv == 0, "jl_flash_prefill: nh=%d not a multiple of nkv=%d", nh, nkv);
   JL_CHECK_ARG(start >= 0 && start + S <= T, "jl_flash_prefill: start=%d + S=%d exceeds cache capacity %d", start, S, T);
@@ -696,7 +713,7 @@ static int flash_launch(const void* q, const void* k_cache, const void* v_cache,
   if (rc) return rc;
   FlashParams p{(__nv_bfloat16*)out, pad_left, B, S, nh, nkv, T, start, scale * 1.4426950408889634f,
                 chunk, sink, sink_logit, gate, ldg, vcos, vsin, v_max_pos, window, softcap * 1.4426950408889634f,
-                softcap > 0.0f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.0f};
+                softcap > 0.0f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.0f, gate_cols};
   dim3 grid((S + FA_BM - 1) / FA_BM, nh, B);
   if (use_v1) {
     const size_t smem = 6 * FA_TILE_BYTES + 128 + 1024;

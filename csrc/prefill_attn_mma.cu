@@ -33,11 +33,11 @@ struct PrefillMmaParams {
   int S, nh, nkv, T, start;
   float scale_log2;
   // the MASKED instances (all off when zero / null): window, blocks of `chunk` positions, capped scores (as in flash_prefill.cu),
-  // a sink in the denominator (logit per head, or 0), a sigmoid gate per (token, head)
+  // a sink in the denominator (logit per head, or 0), a sigmoid gate per (token, head) or, with gate_cols, per (token, channel)
   int window, chunk;
   float cap_log2, cap_rate;
   int sink; const float* sink_logit;
-  const float* gate; int ldg;
+  const float* gate; int ldg; int gate_cols;
 };
 
 __device__ __forceinline__ void pm_mma(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
@@ -201,7 +201,29 @@ __global__ void __launch_bounds__(PM_WARPS * 32) prefill_attn_mma_kernel(const P
     if (l[1] > 0.f) l[1] += exp2f(z - m[1]);
   }
   float inv0 = l[0] > 0.f ? 1.f / l[0] : 0.f, inv1 = l[1] > 0.f ? 1.f / l[1] : 0.f;
-  if (MASKED && p.gate != nullptr) {
+  if (MASKED && p.gate != nullptr && p.gate_cols) {            // tile e: columns 16 t + e (c0, c2) and 16 t + 8 + e (c1, c3) of a half
+#pragma unroll
+    for (int hh = 0; hh < VH; ++hh) {
+      const int col = h * HD + 64 * hh + 16 * t;
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int r = half ? r1 : r0;
+        if (r >= p.S) continue;
+        const float4* g4 = reinterpret_cast<const float4*>(p.gate + ((size_t)b * p.S + r) * p.ldg + col);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const float4 gv = __ldg(g4 + k);
+          const float gs[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const int c = 4 * k + i;                     // column 16 t + c
+            float& v = o[hh][c & 7][2 * half + (c >> 3)];
+            v = __fdividef(v, 1.0f + __expf(-gs[i]));
+          }
+        }
+      }
+    }
+  } else if (MASKED && p.gate != nullptr) {
     if (r0 < p.S) inv0 *= 1.0f / (1.0f + __expf(-p.gate[((size_t)b * p.S + r0) * p.ldg + h]));
     if (r1 < p.S) inv1 *= 1.0f / (1.0f + __expf(-p.gate[((size_t)b * p.S + r1) * p.ldg + h]));
   }
@@ -257,13 +279,15 @@ extern "C" JL_API int jl_prefill_attn_mma(const void* q, const void* k_cache, co
 extern "C" JL_API int jl_prefill_attn_mma_masked(const void* q, const void* k_cache, const void* v_cache, const int* pad_left, void* out,
                                                  int B, int S, int nh, int nkv, int hd, int T, int start, float scale, int window,
                                                  int chunk, float softcap, int sink, const float* sink_logit, const float* gate,
-                                                 int ldg, void* stream) {
+                                                 int ldg, int gate_cols, void* stream) {
   JL_CHECK_ARG(hd == 64, "jl_prefill_attn_mma_masked: head_dim=%d (64 is built)", hd);
   JL_CHECK_ARG(window >= 0 && chunk >= 0 && softcap >= 0.0f && (sink_logit == nullptr || sink) && (gate == nullptr || ldg >= nh),
                "jl_prefill_attn_mma_masked: window %d, chunk %d, softcap %f", window, chunk, softcap);
+  JL_CHECK_ARG(!gate_cols || (gate != nullptr && ldg >= nh * hd && ldg % 4 == 0 && (uintptr_t)gate % 16 == 0),
+               "jl_prefill_attn_mma_masked: a gate per channel needs 16-byte rows (pitch %d)", ldg);
   PrefillMmaParams p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, pad_left,
                      (__nv_bfloat16*)out, S, nh, nkv, T, start, scale * 1.4426950408889634f, window, chunk,
                      softcap * 1.4426950408889634f, softcap > 0.0f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.0f, sink,
-                     sink_logit, gate, ldg};
+                     sink_logit, gate, ldg, gate_cols};
   return mma_launch(p, B, hd, true, stream);
 }

@@ -9,14 +9,14 @@ namespace jl {
 
 template <typename T>
 __global__ void embed_f32_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out, int W,
-                                 int V) {
+                                 int V, float scale) {
   pdl_wait();                      // programmatic dependent launch: nothing is read before the predecessor is done
   pdl_launch_dependents();
   const int m = blockIdx.x;
   int id = ids[m];
   id = id < 0 ? 0 : (id >= V ? V - 1 : id);
   const T* row = table + (size_t)id * W;
-  for (int i = threadIdx.x; i < W; i += blockDim.x) out[(size_t)m * W + i] = to_f(row[i]);
+  for (int i = threadIdx.x; i < W; i += blockDim.x) out[(size_t)m * W + i] = to_f(row[i]) * scale;
 }
 
 // out[m, :] = x[m, :] / sqrt(mean(x^2) + eps) * (offset + w)
@@ -384,9 +384,9 @@ extern "C" JL_API int jl_act_inplace(void* data, int ld, int M, int N, int act, 
   return JL_OK;
 }
 
-extern "C" JL_API int jl_embed_f32(const int* ids, const void* table, float* out, int M, int W, int V, int dtype, void* stream) {
+extern "C" JL_API int jl_embed_f32(const int* ids, const void* table, float* out, int M, int W, int V, float scale, int dtype, void* stream) {
   JL_CHECK_ARG(M >= 1 && W >= 1 && V >= 1, "jl_embed_f32: bad shape M=%d W=%d V=%d", M, W, V);
-  JL_DISPATCH_DTYPE(dtype, JL_LAUNCH_PDL(embed_f32_kernel<T>, dim3(M), dim3(128), 0, (cudaStream_t)stream, ids, (const T*)table, out, W, V));
+  JL_DISPATCH_DTYPE(dtype, JL_LAUNCH_PDL(embed_f32_kernel<T>, dim3(M), dim3(128), 0, (cudaStream_t)stream, ids, (const T*)table, out, W, V, scale));
   JL_CUDA(cudaGetLastError());
   return JL_OK;
 }

@@ -263,8 +263,8 @@ int jl_nvls_selftest(void* mc, const void* src, void* out, int n, int op, unsign
  * stream).  `dtype` 0 = bfloat16, 1 = true float32 (operands, cache and outputs; statistics and sums are fp32 in both).
  * These designs have no counterpart in the reference; the mechanisms are described at the kernels. */
 
-/* ids int32 [M]; table [V, W] of dtype; out fp32 [M, W]. */
-int jl_embed_f32(const int* ids, const void* table, float* out, int M, int W, int V, int dtype, void* stream);
+/* out[m] = scale * table[ids[m]]: ids int32 [M]; table [V, W] of dtype; out fp32 [M, W]. */
+int jl_embed_f32(const int* ids, const void* table, float* out, int M, int W, int V, float scale, int dtype, void* stream);
 /* out[m] = x[m] / sqrt(mean(x[m]^2) + eps) * (offset + w); x fp32 [M, W]; w, out of dtype. */
 int jl_norm_f32(const float* x, const void* w, void* out, int M, int W, float eps, float offset, int dtype, void* stream);
 /* x[m] += norm(y[m]) * (offset + w_post) with y fp32 [M, W] (row pitch ldy); if w_next: h[m] = norm(x[m]) * (offset + w_next). */
@@ -337,7 +337,7 @@ int jl_attn_windowed(const void* q, const void* k_cache, const void* v_cache, vo
  * out32: fp32 output [B*S, H, Dv] written instead of `out`. */
 /* Latent attention, preparation.  y fp32 [B*S, ldy] holds the query latent (q_rank columns at q_off; 0: none) and the key /
  * value latent followed by the rotated key part shared by the heads (kv_rank + rot_dim columns at kv_off).  The latents are
- * RMS-normed with plain weights; the key part is rotated on its first `rot` channels.  cq [B*S, q_rank]; cache
+ * RMS-normed with plain weights (wq_norm NULL: the query columns are brought into dtype as they are); the key part is rotated on its first `rot` channels.  cq [B*S, q_rank]; cache
  * [B][T_cap][kv_rank + rot_dim], the token's row at slot *cache_len + s; c_out [B*S, kv_rank] / kr_out [B*S, rot_dim]
  * (optional): token-major copies of the two parts of the appended row. */
 int jl_latent_prep(const float* y, int ldy, int q_off, int q_rank, int kv_off, int kv_rank, int rot_dim, int rot, int layout,
@@ -422,6 +422,12 @@ size_t jl_delta_scan_ws_floats(int B, int S, int H, int D, int Dv);
 int jl_delta_scan(const float* u, int ldu, int q_off, int k_off, int v_off, int G, const float* y, int ldy, int b_off, int a_off,
                   const void* a2, const void* a_bias, const void* a_log, float* state, float* o, const int* cache_len,
                   const int* pad_left, int B, int S, int H, int D, int Dv, int R, float* ws, int dtype, void* stream);
+/* The same with one decay per head: a_t = exp(-exp(a_log[h]) * softplus(y[m, a_off + h] + a_bias[h])), a_bias and a_log [H]; prompts take
+ * the tokens in blocks of four.  ws: jl_delta_head_scan_ws_floats floats (NULL up to eight tokens per row). */
+size_t jl_delta_head_scan_ws_floats(int B, int S, int H, int G, int D, int Dv);
+int jl_delta_head_scan(const float* u, int ldu, int q_off, int k_off, int v_off, int G, const float* y, int ldy, int b_off, int a_off,
+                       const void* a_bias, const void* a_log, float* state, float* o, const int* cache_len, const int* pad_left, int B,
+                       int S, int H, int D, int Dv, float* ws, int dtype, void* stream);
 
 /* ---- Pieces added with the looped chunked-attention design (Datozen): learned positions, a per-layer token input, attention
  * with a weighted q / k norm before the rotation, rotated values, blocks of positions and a learned sink, a router with a
@@ -443,35 +449,38 @@ int jl_branch_add_cast(const float* y1, int ld1, const float* y2, int ld2, float
                        void* stream);
 /* jl_attn_prep with: `layout` of the rotated q / k pairs (0: (2i, 2i+1), 1: (i, i + rot/2)); q_norm_w / k_norm_w [D] of dtype, an RMS
  * norm of every head before the rotation (NULL: none); v_cos / v_sin fp32 [v_max_pos][Dv/2]: values rotated at their own position
- * over all Dv channels before they are cached, pairs as v_layout (NULL: cached as they are). */
+ * over all Dv channels before they are cached, pairs as v_layout (NULL: cached as they are); q_every > 0: the finished query is
+ * multiplied by 1 + q_coef * ln(1 + floor((position + 1) / q_every)). */
 int jl_attn_prep_ex(const float* y, int ldy, int q_off, int k_off, int v_off, void* q_out, void* k_cache, void* v_cache,
                     const float* cos_t, const float* sin_t, int max_pos, int rot, int layout, int unit_norm, const void* q_norm_w,
                     const void* k_norm_w, float eps, const float* v_cos, const float* v_sin, int v_max_pos, int v_layout,
                     const int* cache_len, const int* pad_left, int B, int S, int H, int G, int D, int Dv, int T_cap,
-                    const float* bias, int v_norm, int v_token_major, int dtype, void* stream);
-/* jl_attn_windowed with: gate (fp32 pre-activation of a sigmoid per head, column h of row m, pitch ldg; NULL: none); chunk > 0:
+                    const float* bias, int v_norm, int v_token_major, float q_coef, int q_every, int dtype, void* stream);
+/* jl_attn_windowed with: gate (fp32 pre-activation of a sigmoid per head, column h of row m, or with gate_cols one per channel, column
+ * h * Dv + c; pitch ldg; NULL: none); chunk > 0:
  * positions form blocks of `chunk` and a query sees the keys of its own block only; softcap > 0: scores become softcap *
  * tanh(score / softcap); sink_logit fp32 [H]: the extra term of the
  * denominator is exp(sink_logit[h]) (needs sink = 1; NULL: exp(0)); v_cos / v_sin: the cached values were rotated at their own
  * positions and every head's sum is rotated back by the query's position before the gate. */
-int jl_attn_masked(const void* q, const void* k_cache, const void* v_cache, void* out, const float* gate, int ldg,
+int jl_attn_masked(const void* q, const void* k_cache, const void* v_cache, void* out, const float* gate, int ldg, int gate_cols,
                    const int* cache_len, const int* pad_left, int B, int S, int H, int G, int D, int Dv, int T_cap, int ldk, int ldv,
                    long long k_bs, long long k_hs, long long v_bs, long long v_hs, int window, int chunk, float scale, float softcap,
                    float* scratch, int splits, int sink, const float* sink_logit, const float* v_cos, const float* v_sin, int v_max_pos,
                    int v_layout, float* out32, int dtype, void* stream);
 /* The tcgen05 prompt attention kernel (bfloat16, 128-wide heads; caches [B, nkv, T, 128]) with blocks of `chunk` positions, a sink in
- * the denominator (sink_logit fp32 [nh] or NULL for exp(0)), a sigmoid gate per (token, head) (fp32 pre-activation, pitch ldg) and the
+ * the denominator (sink_logit fp32 [nh] or NULL for exp(0)), a sigmoid gate per (token, head) (fp32 pre-activation, pitch ldg; with
+ * gate_cols one per channel, column h * hd + d, rows on 16-byte boundaries) and the
  * turn back of values cached rotated at their own positions (v_cos / v_sin fp32 [v_max_pos][64], pairs m, m + 64).  `start`: slots
  * filled before this call's S tokens per row.  window > 0: a query sees itself and the window - 1 slots before it; softcap > 0: scores
  * become softcap * tanh(score / softcap).  hd = 64 (without rotated values) runs jl_prefill_attn_mma_masked. */
 int jl_flash_prefill_masked(const void* q, const void* k_cache, const void* v_cache, const int* pad_left, void* out, int B, int S,
                             int nh, int nkv, int hd, int T, int start, float scale, int chunk, int sink, const float* sink_logit,
-                            const float* gate, int ldg, const float* v_cos, const float* v_sin, int v_max_pos, int window,
-                            float softcap, void* stream);
+                            const float* gate, int ldg, int gate_cols, const float* v_cos, const float* v_sin, int v_max_pos,
+                            int window, float softcap, void* stream);
 /* jl_prefill_attn_mma (hd = 64) with the same options, values as they are. */
 int jl_prefill_attn_mma_masked(const void* q, const void* k_cache, const void* v_cache, const int* pad_left, void* out, int B, int S,
                                int nh, int nkv, int hd, int T, int start, float scale, int window, int chunk, float softcap, int sink,
-                               const float* sink_logit, const float* gate, int ldg, void* stream);
+                               const float* sink_logit, const float* gate, int ldg, int gate_cols, void* stream);
 /* jl_moe_route with: choice_bias fp32 [E] added to the scores for the choice (group scores and top) only; experts n_real .. E-1
  * are identity experts: a chosen one is reported as expert -1 (jl_moe_sort and the grouped linears skip it) and its weight is
  * added to ident_w[m]. */

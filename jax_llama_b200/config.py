@@ -16,7 +16,7 @@ import json
 import logging
 import os
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional, Union
+from typing import Any, Dict, List, Optional, Tuple, Union
 
 logger = logging.getLogger(__name__)
 
@@ -320,6 +320,9 @@ class AttentionMixerSpec:
     v_from_k: bool = False          # no value projection: the values are the keys before norm and rotation
     v_mix: str = ""                 # "first": this layer's values are kept for the step; "mix": v <- (1 - vmix) v + vmix v_first
     out_bias: bool = False          # the output projection has a bias (`o.b`)
+    channel_gate: bool = False      # `g` [heads · vdim]: one sigmoid gate per output channel (instead of head_gate's one per head)
+    q_growth: Optional[Tuple[float, int]] = None   # (coef, every): the finished query at position p is multiplied by
+                                    # 1 + coef · ln(1 + floor((p + 1) / every))
     kind: str = "attention"
 
 
@@ -335,10 +338,11 @@ class GlaMixerSpec:
 
 @dataclass
 class LatentAttentionMixerSpec:
-    """Softmax attention through low-rank latents: queries from a normed latent of size q_rank, keys and values from a
-    normed latent of size kv_rank (what the layer caches, with one rotated key part of rot_dim channels shared by the
-    heads).  A head's query / key is `dim` unrotated channels followed by `rot_dim` rotated ones; `window` > 0 limits a
-    query to the last `window` positions up to its own."""
+    """Softmax attention through low-rank latents: queries from a normed latent of size q_rank (0: projected directly, `q`),
+    keys and values from a normed latent of size kv_rank (what the layer caches, with one rotated key part of rot_dim channels
+    shared by the heads).  A head's query / key is `dim` unrotated channels followed by `rot_dim` rotated ones; `window` > 0
+    limits a query to the last `window` positions up to its own.  sink_learned: one more term exp(sink[head]) in the softmax
+    denominator; head_gate: one sigmoid gate per head on the output."""
     heads: int
     dim: int
     rot_dim: int
@@ -348,6 +352,8 @@ class LatentAttentionMixerSpec:
     scale: float
     rot: Optional[RotarySpec] = None
     window: int = 0
+    sink_learned: bool = False
+    head_gate: bool = False
     kind: str = "latent_attention"
 
 
@@ -380,14 +386,16 @@ class StateSpaceMixerSpec:
 
 @dataclass
 class DeltaMixerSpec:
-    """Gated delta rule with one decay per key channel: S <- diag(a) S; e = beta (v - Sᵀk); S <- S + k eᵀ; o = Sᵀq.
-    q / k heads (kv_heads of `dim`) shared by groups of value heads, each of q, k, v through a causal convolution of
-    `conv` taps and silu, q and k scaled to unit length; read-out normed per head and gated by a low-rank sigmoid gate."""
+    """Gated delta rule: S <- diag(a) S; e = beta (v - Sᵀk); S <- S + k eᵀ; o = Sᵀq.  q / k heads (kv_heads of `dim`) shared by
+    groups of value heads, each of q, k, v through a causal convolution of `conv` taps and silu, q and k scaled to unit length.
+    head_decay False: one decay per key channel from a low-rank projection (`a1`, `a2`), read-out normed per head and gated by a
+    low-rank sigmoid gate (`g1`, `g2`); True: one decay per head (`a`), a full silu gate (`g`)."""
     heads: int
     kv_heads: int
     dim: int
     vdim: int
     conv: int = 4
+    head_decay: bool = False
     kind: str = "channel_delta"
 
 
@@ -515,6 +523,7 @@ class HybridConfig:
         self.logit_softcap = float(logit_softcap) if logit_softcap else 0.0
         self.residual_mult = float(residual_mult)
         self.embedding_dict = copy.deepcopy(embedding) if embedding else None
+        self.embedding_scale = float((embedding or {}).get("scale", 1.0))       # factor on the token embedding's rows
         bg = (embedding or {}).get("bigram")
         self.pair_embedding = PairEmbeddingSpec(int(bg["buckets"]), int(bg["mul_prev"]), int(bg["mul_cur"])) if bg else None
         # layers [start, stop) run `times` times in a row with the same weights (every pass has its own cache and state)
@@ -944,3 +953,78 @@ class KetolixConfig(HybridConfig):
                 raise ValueError(f"layer {i}: {len(m.right.decay)} decays for {m.right.heads} heads")
         if m.kind == "mlstm" and m.gate_cap <= 0:
             raise ValueError(f"layer {i}: gate_cap must be positive")
+
+
+class FiponexConfig(HybridConfig):
+    """Fiponex: a decoder of sandwich blocks — every sublayer between a zero-centred RMS norm before and one after — over a scaled
+    token embedding, with a head of its own.
+
+    Mixers: "attention" — grouped heads without rotation; q, k and v with biases; q and k normed per head with a weight; queries
+    that grow slowly with their position; a learned logit per head in the softmax denominator; one sigmoid gate per output channel.
+    "latent_attention" — queries projected directly, keys and values from one normed latent per token with a rotated key part
+    shared by the heads; sliding window; a learned logit per head in the softmax denominator; a sigmoid gate per head.  "delta" —
+    gated delta rule with one decay per head over convolved q, k and v, a full silu gate.  Feed-forward: a relu-gated dense layer or
+    a mixture of silu-gated experts weighted by their softmax scores as they are.
+
+    ``config.json``: ``vocab``, ``width``, ``norm.eps``, ``embedding.scale`` and ``layers[i]`` = ``{type, mixer, mlp}`` with, for
+    "attention", ``mixer.{heads, kv_heads, dim, vdim, scale, q_temp.{coef, every}}``; for "latent_attention", ``mixer.{heads, dim,
+    rot_dim, vdim, kv_rank, scale, mask.size, rot.{dims, base}}``; for "delta", ``mixer.{heads, kv_heads, dim, vdim, conv}``; ``mlp``
+    null, ``{kind: dense, ff}`` or ``{kind: moe, router.{experts, top}, expert.ff}``."""
+
+    model_type = "fiponex"
+    architecture = "Fiponex"
+    block = "sandwich"
+    norm_offset = 1.0
+
+    def _parse_mixer(self, i: int, d: Dict[str, Any]) -> Any:
+        m = d["mixer"]
+        kind = d["type"]
+        if kind == "attention":
+            t = m.get("q_temp")
+            if t and float(t["every"]) != int(t["every"]):
+                raise ValueError(f"layer {i}: q_temp.every {t['every']} is not a whole number of positions")
+            return AttentionMixerSpec(
+                heads=int(m["heads"]), kv_heads=int(m.get("kv_heads", m["heads"])), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                scale=float(m["scale"]), rot=None, kv_from=None, qk_unit_norm=False, head_gate=False, channel_gate=True, bias=True,
+                qk_norm=True, sink=True, sink_learned=True, q_growth=(float(t["coef"]), int(t["every"])) if t else None)
+        if kind == "latent_attention":
+            return LatentAttentionMixerSpec(
+                heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]), q_rank=0,
+                kv_rank=int(m["kv_rank"]), scale=float(m["scale"]), rot=RotarySpec.parse(m.get("rot"), "interleaved"),
+                window=int((m.get("mask") or {}).get("size") or 0), sink_learned=True, head_gate=True)
+        if kind == "delta":
+            return DeltaMixerSpec(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads", m["heads"])), dim=int(m["dim"]),
+                                  vdim=int(m["vdim"]), conv=int(m["conv"]), head_decay=True, kind="delta")
+        raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+
+    def _parse_mlp(self, i: int, mlp: Optional[Dict[str, Any]]) -> Any:
+        if mlp is None:
+            return None
+        kind = mlp.get("kind", "dense")
+        if kind == "dense":
+            return DenseMlpSpec(ff=int(mlp["ff"]), act="relu", gated=True)
+        if kind == "moe":
+            r = mlp["router"]
+            return MoeMlpSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(mlp["expert"]["ff"]), act="silu", score="softmax",
+                              groups=1, keep=1, scale=1.0, normalise=False, gated=True)
+        raise ValueError(f"layer {i}: unknown feed-forward kind {kind!r}")
+
+    def _validate_layer(self, i: int, l: HybridLayerSpec) -> None:
+        m = l.mixer
+        if m.kind == "latent_attention":
+            if min(m.heads, m.dim + m.rot_dim, m.vdim, m.kv_rank) <= 0 or min(m.dim, m.rot_dim, m.window) < 0:
+                raise ValueError(f"layer {i}: latent attention sizes heads {m.heads}, dim {m.dim} + {m.rot_dim}, window {m.window}")
+            if m.rot is not None and (m.rot.dims % 2 or m.rot.dims > m.rot_dim):
+                raise ValueError(f"layer {i}: rot.dims {m.rot.dims} must be even and at most rot_dim {m.rot_dim}")
+            if m.rot_dim > 0 and m.rot is None:
+                raise ValueError(f"layer {i}: rot_dim {m.rot_dim} without rot")
+        else:
+            if min(m.heads, m.kv_heads, m.dim, m.vdim) <= 0 or m.heads % m.kv_heads:
+                raise ValueError(f"layer {i}: {m.kind} sizes heads {m.heads}, kv_heads {m.kv_heads}, {m.dim} / {m.vdim}")
+            if m.kind == "attention" and m.q_growth is not None and m.q_growth[1] < 1:
+                raise ValueError(f"layer {i}: q_temp.every {m.q_growth[1]} must be at least 1")
+            if m.kind == "delta" and not 1 <= m.conv <= 32:
+                raise ValueError(f"layer {i}: {m.conv} taps")
+        f = l.mlp
+        if f is not None and f.kind == "moe" and not 1 <= f.top <= f.experts:
+            raise ValueError(f"layer {i}: top {f.top} of {f.experts} experts")

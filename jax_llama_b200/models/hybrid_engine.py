@@ -160,12 +160,6 @@ def tensor_shapes(config: Any, decay_rank: int = 16, present: Optional[Dict[str,
             out.update({p + "mix.q": (m.heads * m.dim, W), p + "mix.k": (m.heads * m.dim, W),
                         p + "mix.v": (m.heads * m.vdim, W), p + "mix.g": (m.heads * m.vdim, W),
                         p + "mix.o": (W, m.heads * m.vdim)})
-        elif m.kind == "latent_attention":
-            out.update({p + "mix.dq": (m.q_rank, W), p + "mix.dq.norm": (m.q_rank,),
-                        p + "mix.uq": (m.heads * (m.dim + m.rot_dim), m.q_rank),
-                        p + "mix.dkv": (m.kv_rank + m.rot_dim, W), p + "mix.dkv.norm": (m.kv_rank,),
-                        p + "mix.uk": (m.heads * m.dim, m.kv_rank), p + "mix.uv": (m.heads * m.vdim, m.kv_rank),
-                        p + "mix.o": (W, m.heads * m.vdim)})
         else:
             out[p + "mix.q"] = (m.heads * m.dim, W)
             if m.kv_from is None:
@@ -234,6 +228,9 @@ class HybridEngine(B200Engine):
         self.side_table = get("side.embed") if config.token_side_dim else None
         if (self.pos_table is not None or self.side_table is not None) and (self.pair_table is not None or config.embed_norm):
             raise ValueError("learned positions and token inputs do not combine with a pair-hash or normed embedding")
+        self.embed_scale = float(config.embedding_scale)
+        if self.embed_scale != 1.0 and (self.pair_table is not None or config.embed_norm or self.pos_table is not None):
+            raise ValueError("a scaled embedding does not combine with pair-hash, normed or position embeddings")
         if self.side_table is not None and not self.parallel:
             raise ValueError("per-layer token inputs go with parallel blocks")
         if self.pair_table is None and self.embed_norm is not None:
@@ -375,7 +372,7 @@ class HybridEngine(B200Engine):
             ids = self._step_ids(ids, cache)
         if self.pos_table is not None:
             return SK.embed_pos(ids, self.embedding, self.pos_table, cache.len_dev, cache.pad_left, B, S, out=out)
-        return SK.embed_f32(ids, self.embedding, out=out)
+        return SK.embed_f32(ids, self.embedding, out=out, scale=self.embed_scale)
 
     def _head(self, x: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         c = self.config
@@ -518,7 +515,7 @@ def random_tensors(config: Any, device: Any = "cuda", seed: int = 0, decay_rank:
         return torch.randn(shape, generator=g, device=dev, dtype=torch.float32)
 
     for name, shape in tensor_shapes(config, decay_rank).items():
-        if name.endswith("mix.norm") or name.endswith("right.norm") or (config.norm_offset == 0.0 and len(shape) == 1 and "norm" in name):
+        if (".mix." in name and name.endswith("norm")) or (config.norm_offset == 0.0 and len(shape) == 1 and "norm" in name):
             t = 1.0 + 0.1 * randn(shape)
         elif name.endswith("mix.a2.b"):
             t = 2.0 + 2.0 * randn(shape)

@@ -133,7 +133,8 @@ class AttentionMixer(Mixer):
     And: an RMS norm over all heads of q (of k) together (`qk_norm_all`); scores capped by tanh (`softcap`); a causal convolution on q
     and k behind the projection (`conv`, its last inputs are state), values that are the convolved keys (`v_from_k`); values mixed
     with those of the first such layer (`v_mix`: that layer leaves a view of its fp32 values with the cache for the step, the
-    mixed value is what later layers cache); a bias on the output projection (`out_bias`)."""
+    mixed value is what later layers cache); a bias on the output projection (`out_bias`); one sigmoid gate per output channel
+    (`channel_gate`), applied where the attention kernels store their result; queries that grow with their position (`q_growth`)."""
 
     kind = "attention"
 
@@ -141,10 +142,11 @@ class AttentionMixer(Mixer):
         self.spec, self.eps = spec, float(eps)
         self.shares_kv = spec.kv_from is not None
         own = [] if self.shares_kv else [w["k"]] if spec.v_from_k else [w["k"], w["v"]]
-        self.w_in, offs = _stack_rows([w["q"]] + own + ([w["g"]] if spec.head_gate else []))
+        self.gates = spec.heads * spec.vdim if spec.channel_gate else spec.heads if spec.head_gate else 0
+        self.w_in, offs = _stack_rows([w["q"]] + own + ([w["g"]] if self.gates else []))
         self.q_off = offs[0]
         self.k_off, self.v_off = (-1, -1) if self.shares_kv else (offs[1], offs[1] if spec.v_from_k else offs[2])
-        self.g_off = offs[-1] if spec.head_gate else -1
+        self.g_off = offs[-1] if self.gates else -1
         self.wo = w["o"].contiguous()
         self.dtype = self.wo.dtype
         self._decode_plans: Dict[Tuple[int, int], Tuple[int, Optional[torch.Tensor]]] = {}
@@ -155,10 +157,15 @@ class AttentionMixer(Mixer):
                 if off >= 0 and name + ".b" in w:
                     self.bias[off:off + w[name].shape[0]] = w[name + ".b"].float()
         self.talk = w["talk"].contiguous() if spec.talking_heads else None
-        if spec.talking_heads and (self.shares_kv or spec.head_gate):
-            raise ValueError("mixed attention weights go with a layer's own keys / values and no head gate")
+        if spec.talking_heads and (self.shares_kv or self.gates):
+            raise ValueError("mixed attention weights go with a layer's own keys / values and no output gate")
+        if spec.channel_gate and (spec.head_gate or spec.v_rot):
+            raise ValueError("a gate per channel goes with values as they are and no gate per head")
+        if spec.q_growth is not None and spec.qk_norm_all:
+            raise ValueError("growing queries go with norms per head (or none)")
         self.plain = not (spec.bias or spec.v_unit_norm or spec.window or spec.sink or spec.talking_heads or spec.qk_norm
                           or spec.chunk or spec.v_rot or spec.softcap or spec.qk_norm_all or spec.conv or spec.v_from_k
+                          or spec.channel_gate or spec.q_growth is not None
                           or (spec.rot is not None and spec.rot.layout != "interleaved"))
         any_norm = spec.qk_norm or spec.qk_norm_all
         self.q_norm = w["q.norm"].contiguous() if any_norm else None
@@ -187,8 +194,8 @@ class AttentionMixer(Mixer):
             out["k"] = (spec.kv_heads * spec.dim, W)
             if not spec.v_from_k:
                 out["v"] = (spec.kv_heads * spec.vdim, W)
-        if spec.head_gate:
-            out["g"] = (spec.heads, W)
+        if spec.head_gate or spec.channel_gate:
+            out["g"] = (spec.heads * (spec.vdim if spec.channel_gate else 1), W)
         if spec.conv:
             out["q.conv"], out["k.conv"] = (spec.heads * spec.dim, spec.conv), (spec.kv_heads * spec.dim, spec.conv)
         if spec.v_mix:
@@ -271,10 +278,11 @@ class AttentionMixer(Mixer):
                          None if self.shares_kv else vc, rope[0], rope[1], rot, s.qk_unit_norm, self.eps, cache.len_dev,
                          cache.pad_left, B, S, s.heads, s.kv_heads, s.dim, s.vdim, bias=self.bias, v_unit_norm=s.v_unit_norm,
                          v_token_major=s.talking_heads, layout=layout, q_norm_w=self.q_norm,
-                         k_norm_w=self.k_norm if self.k_norm is not None else self.q_norm, v_cos=v_cos, v_sin=v_sin)
+                         k_norm_w=self.k_norm if self.k_norm is not None else self.q_norm, v_cos=v_cos, v_sin=v_sin,
+                         q_growth=s.q_growth)
         if s.talking_heads:
             return self._attend_mixed(q, kc, vc, cache, B, S)
-        gate = y[:, self.g_off:self.g_off + s.heads] if s.head_gate else None
+        gate = y[:, self.g_off:self.g_off + self.gates] if self.gates else None
         if not self.plain and (gate is not None or s.chunk or s.sink_learned or s.v_rot or s.softcap):
             if S > 1 and self._flash_masked_shape():
                 # prompts of 128-wide heads in bfloat16: the tcgen05 kernel with the block bound, the window, the cap, the sink, the
@@ -283,7 +291,7 @@ class AttentionMixer(Mixer):
                 _lib.check(_lib.lib().jl_flash_prefill_masked(
                     q.data_ptr(), kc.data_ptr(), vc.data_ptr(), cache.pad_left.data_ptr(), out.data_ptr(), B, S, s.heads,
                     s.kv_heads, s.dim, kc.shape[2], int(cache.index), float(s.scale), int(s.chunk), int(s.sink),
-                    K._p(self.sink_logit), K._p(gate), gate.stride(0) if gate is not None else 0, K._p(v_cos), K._p(v_sin),
+                    K._p(self.sink_logit), K._p(gate), gate.stride(0) if gate is not None else 0, int(s.channel_gate), K._p(v_cos), K._p(v_sin),
                     v_cos.shape[0] if v_cos is not None else 0, int(s.window), float(s.softcap), K._stream()),
                     "jl_flash_prefill_masked")
                 return out
@@ -407,19 +415,29 @@ class LatentAttentionMixer(Mixer):
     with per-head keys [k_rot | U_h c] and values V_h c in token-major layout, which costs a third of the arithmetic of
     the latent-space form at these head sizes.  Both forms run the windowed generic attention kernel.
 
-    Internally a query head is laid out [rot_dim rotated | dim unrotated] (the rows of the query up-projection are
-    permuted once at load), so that the rotation applies to the leading channels of a head as in the other mixers."""
+    Internally a query head is laid out [rot_dim rotated | dim unrotated] (the rows of the query (up-)projection are
+    permuted once at load), so that the rotation applies to the leading channels of a head as in the other mixers.
+
+    Options of the spec: queries projected directly instead of through a latent (q_rank 0: their projection joins the stacked one
+    and the preparation kernel brings them into the operand type), a learned sink logit per head, a sigmoid gate per head (a scalar
+    per head, so in latent space it is applied before the values' up-projection, where the attention kernel stores)."""
 
     kind = "latent_attention"
 
     def __init__(self, spec: LatentAttentionMixerSpec, w: Dict[str, torch.Tensor], eps: float):
         self.spec, self.eps = spec, float(eps)
         s = spec
-        self.w_in, offs = _stack_rows([w["dq"], w["dkv"]])
-        self.q_off, self.kv_off = offs
-        self.q_norm, self.kv_norm = w["dq.norm"].contiguous(), w["dkv.norm"].contiguous()
-        uq = w["uq"].view(s.heads, s.dim + s.rot_dim, s.q_rank)                 # stored [dim unrotated | rot_dim rotated]
-        self.uq = torch.cat([uq[:, s.dim:], uq[:, :s.dim]], 1).reshape(s.heads * (s.dim + s.rot_dim), s.q_rank).contiguous()
+        qn = s.heads * (s.dim + s.rot_dim)
+        wq = w["uq" if s.q_rank else "q"]
+        wq = wq.view(s.heads, s.dim + s.rot_dim, wq.shape[1])                   # stored [dim unrotated | rot_dim rotated]
+        wq = torch.cat([wq[:, s.dim:], wq[:, :s.dim]], 1).reshape(qn, wq.shape[2]).contiguous()
+        self.uq = wq if s.q_rank else None
+        self.q_cols = s.q_rank or qn                                            # query columns of the stacked projection
+        self.w_in, offs = _stack_rows([w["dq"] if s.q_rank else wq, w["dkv"]] + ([w["g"]] if s.head_gate else []))
+        self.q_off, self.kv_off = offs[:2]
+        self.g_off = offs[2] if s.head_gate else -1
+        self.q_norm, self.kv_norm = w["dq.norm"].contiguous() if s.q_rank else None, w["dkv.norm"].contiguous()
+        self.sink_logit = w["sink"].float().contiguous() if s.sink_learned else None
         self.uk_t = w["uk"].view(s.heads, s.dim, s.kv_rank).transpose(1, 2).contiguous()    # [H, kv_rank, dim]
         self.uv = w["uv"].view(s.heads, s.vdim, s.kv_rank).contiguous()          # [H, vdim, kv_rank]
         self.w_kv, kv_offs = _stack_rows([w["uk"], w["uv"]])                     # [H·dim | H·vdim, kv_rank]: prompts
@@ -430,7 +448,34 @@ class LatentAttentionMixer(Mixer):
 
     def weights(self) -> List[torch.Tensor]:
         """What a decode step streams (the stacked up-projection of prompts holds the same values once more)."""
-        return [self.w_in, self.q_norm, self.kv_norm, self.uq, self.uk_t, self.uv, self.wo]
+        return [self.w_in, self.kv_norm, self.uk_t, self.uv, self.wo] + [t for t in (self.q_norm, self.uq, self.sink_logit)
+                                                                         if t is not None]
+
+    @staticmethod
+    def shapes(spec: LatentAttentionMixerSpec, W: int, rank_of: "object" = None) -> Dict[str, Tuple[int, ...]]:
+        qn = spec.heads * (spec.dim + spec.rot_dim)
+        out: Dict[str, Tuple[int, ...]] = {
+            "dkv": (spec.kv_rank + spec.rot_dim, W), "dkv.norm": (spec.kv_rank,), "uk": (spec.heads * spec.dim, spec.kv_rank),
+            "uv": (spec.heads * spec.vdim, spec.kv_rank), "o": (W, spec.heads * spec.vdim)}
+        if spec.q_rank:
+            out["dq"], out["dq.norm"], out["uq"] = (spec.q_rank, W), (spec.q_rank,), (qn, spec.q_rank)
+        else:
+            out["q"] = (qn, W)
+        if spec.head_gate:
+            out["g"] = (spec.heads, W)
+        if spec.sink_learned:
+            out["sink"] = (spec.heads,)
+        return out
+
+    def _attend(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cache: "object", B: int, S: int, H: int, G: int, D: int,
+                Dv: int, T_cap: int, ldk: int, ldv: int, gate: Optional[torch.Tensor],
+                strides: "Tuple[int, int, int, int]" = (0, 0, 0, 0)) -> torch.Tensor:
+        s = self.spec
+        if gate is None and not s.sink_learned:
+            return SK.attn_windowed(q, k, v, cache.len_dev, cache.pad_left, B, S, H, G, D, Dv, T_cap, ldk, ldv, s.window, s.scale,
+                                    strides=strides)
+        return SK.attn_masked(q, k, v, cache.len_dev, cache.pad_left, B, S, H, G, D, Dv, s.scale, gate=gate, window=s.window,
+                              sink=s.sink_learned, sink_logit=self.sink_logit, T_cap=T_cap, ldk=ldk, ldv=ldv, strides=strides)
 
     def new_cache(self, batch: int, length: int, device: torch.device) -> Tuple[torch.Tensor, None]:
         return torch.zeros((batch, length, self.row), dtype=self.dtype, device=device), None
@@ -446,27 +491,27 @@ class LatentAttentionMixer(Mixer):
         layout = SK.ROT_LAYOUTS[s.rot.layout] if s.rot is not None else 0
         kc = cache.ks[layer]                                                   # [B, T, kv_rank + rot_dim]
         starts = S > 1 and int(cache.index) == 0                               # a prompt from an empty cache
-        y = SK.linear(h, self.w_in)                                            # fp32 [M, query latent | kv latent | key part]
-        cq, c_new, kr_new = SK.latent_prep(y, self.q_off, s.q_rank, self.kv_off, s.kv_rank, s.rot_dim, rot, layout,
+        y = SK.linear(h, self.w_in)                                            # fp32 [M, queries (or latent) | kv latent | key part | gate]
+        gate = y[:, self.g_off:self.g_off + H] if s.head_gate else None
+        cq, c_new, kr_new = SK.latent_prep(y, self.q_off, self.q_cols, self.kv_off, s.kv_rank, s.rot_dim, rot, layout,
                                            self.q_norm, self.kv_norm, kc, rope[0], rope[1], self.eps, cache.len_dev,
                                            cache.pad_left, B, S, token_major=starts)
-        q = SK.linear(cq, self.uq, out_f32=False)                              # [M, H·(rot_dim + dim)]
+        q = SK.linear(cq, self.uq, out_f32=False) if s.q_rank else cq          # [M, H·(rot_dim + dim)]
         if starts:
-            return self._attend_projected(q, c_new, kr_new, cache, B, S, rot, layout, rope)
+            return self._attend_projected(q, c_new, kr_new, cache, B, S, rot, layout, rope, gate)
         qa = torch.empty((M, H * self.row), dtype=self.dtype, device=h.device)
         a = q[:, s.rot_dim:] if s.rot_dim else q                               # head h's unrotated part starts at h·qd
         SK.linear_batched(a, self.uk_t, qa, nbatch=H, rows=M, x_bs=qd, o_bs=self.row)      # U_hᵀ a_h
         if s.rot_dim:
             SK.rotary_slice(q, qd, 0, qa, self.row, s.kv_rank, H, s.rot_dim, rot, layout, rope[0], rope[1],
                             cache.len_dev, cache.pad_left, B, S)
-        ctx = SK.attn_windowed(qa, kc, kc, cache.len_dev, cache.pad_left, B, S, H, 1, self.row, s.kv_rank, kc.shape[1],
-                               self.row, self.row, s.window, s.scale)         # [M, H·kv_rank]
+        ctx = self._attend(qa, kc, kc, cache, B, S, H, 1, self.row, s.kv_rank, kc.shape[1], self.row, self.row, gate)     # [M, H·kv_rank]
         out = torch.empty((M, H * s.vdim), dtype=self.dtype, device=h.device)
         SK.linear_batched(ctx, self.uv, out, nbatch=H, rows=M, x_bs=s.kv_rank, o_bs=s.vdim)
         return out
 
     def _attend_projected(self, q: torch.Tensor, c_new: torch.Tensor, kr_new: torch.Tensor, cache: "object", B: int, S: int,
-                          rot: int, layout: int, rope: Tuple[torch.Tensor, torch.Tensor]) -> torch.Tensor:
+                          rot: int, layout: int, rope: Tuple[torch.Tensor, torch.Tensor], gate: Optional[torch.Tensor]) -> torch.Tensor:
         """Per-head keys and values of the S new tokens of every row, token-major; slot == index within the prompt."""
         s = self.spec
         M, H, qd = B * S, s.heads, s.dim + s.rot_dim
@@ -479,8 +524,7 @@ class LatentAttentionMixer(Mixer):
         SK.rotary_slice(kv, s.dim, 0, kf, qd, s.rot_dim, H, s.dim, 0, 0, rope[0], rope[1], cache.len_dev, cache.pad_left, B, S)
         v = kv[:, self.v_col:]
         ldv = kv.stride(0)
-        return SK.attn_windowed(qf, kf, v, cache.len_dev, cache.pad_left, B, S, H, H, qd, s.vdim, S, H * qd, ldv, s.window,
-                                s.scale, strides=(S * H * qd, qd, S * ldv, s.vdim))
+        return self._attend(qf, kf, v, cache, B, S, H, H, qd, s.vdim, S, H * qd, ldv, gate, strides=(S * H * qd, qd, S * ldv, s.vdim))
 
 
 class RetentionMixer(Mixer):
@@ -575,24 +619,30 @@ class StateSpaceMixer(Mixer):
 
 
 class DeltaRuleMixer(Mixer):
-    """Gated delta rule with one decay per key channel (see `DeltaMixerSpec`).  One stacked projection
-    [q | k | v | beta | decay rank | gate rank]; q, k, v through ONE causal convolution call (their filters stacked; state:
+    """Gated delta rule (see `DeltaMixerSpec`) with one decay per key channel or per head.  One stacked projection
+    [q | k | v | beta | decay rank | gate rank], with one decay per head [q | k | v | gate | beta | decay]; q, k, v through ONE causal convolution call (their filters stacked; state:
     the last taps − 1 inputs) and silu; the scan kernels normalise q / k, form beta and the decays
-    exp(−exp(A_log) softplus(A2 · + bias)) and advance the fp32 state; the read-out is normed per head (weight shared by
-    the heads) and gated by sigmoid of the low-rank gate."""
+    exp(−exp(A_log) softplus(A2 · + bias)) — or exp(−exp(A_log) softplus(a + bias)) — and advance the fp32 state; the read-out is
+    normed per head (weight shared by the heads) and gated by sigmoid of the low-rank gate or silu of the full one."""
 
     kind = "channel_delta"
 
     def __init__(self, spec: DeltaMixerSpec, w: Dict[str, torch.Tensor], eps: float):
         self.spec, self.eps = spec, float(eps)
         s = spec
-        self.w_in, offs = _stack_rows([w["q"], w["k"], w["v"], w["b"], w["a1"], w["g1"]])
-        self.q_off, self.k_off, self.v_off, self.b_off, self.a_off, self.g_off = offs
+        if s.head_decay:
+            self.w_in, offs = _stack_rows([w["q"], w["k"], w["v"], w["g"], w["b"], w["a"]])
+            self.q_off, self.k_off, self.v_off, self.g_off, self.b_off, self.a_off = offs
+        else:
+            self.w_in, offs = _stack_rows([w["q"], w["k"], w["v"], w["b"], w["a1"], w["g1"]])
+            self.q_off, self.k_off, self.v_off, self.b_off, self.a_off, self.g_off = offs
         self.nq, self.nv = s.kv_heads * s.dim, s.heads * s.vdim
         self.conv_w = torch.cat([w["q.conv"], w["k.conv"], w["v.conv"]], 0).contiguous()
-        self.a2, self.a_bias, self.a_log = w["a2"].contiguous(), w["dt_bias"].contiguous(), w["A_log"].contiguous()
-        self.g2 = w["g2"].contiguous()
-        self.gate_rank = w["g1"].shape[0]
+        self.a_bias, self.a_log = w["dt_bias"].contiguous(), w["A_log"].contiguous()
+        self.a2 = self.g2 = None
+        if not s.head_decay:
+            self.a2, self.g2 = w["a2"].contiguous(), w["g2"].contiguous()
+            self.gate_rank = w["g1"].shape[0]
         self.norm = w["norm"].contiguous()
         self.wo = w["o"].contiguous()
         self.dtype = self.wo.dtype
@@ -601,13 +651,15 @@ class DeltaRuleMixer(Mixer):
     def shapes(spec: DeltaMixerSpec, W: int, rank_of: "object" = None) -> Dict[str, Tuple[int, ...]]:
         rank_of = rank_of or (lambda name, default: default)
         nq, nv, nd = spec.kv_heads * spec.dim, spec.heads * spec.vdim, spec.heads * spec.dim
+        out = {"q": (nq, W), "q.conv": (nq, spec.conv), "k": (nq, W), "k.conv": (nq, spec.conv), "v": (nv, W),
+               "v.conv": (nv, spec.conv), "b": (spec.heads, W), "A_log": (spec.heads,), "norm": (spec.vdim,), "o": (W, nv)}
+        if spec.head_decay:
+            return {**out, "a": (spec.heads, W), "dt_bias": (spec.heads,), "g": (nv, W)}
         ra, rg = rank_of("a1", 16), rank_of("g1", 16)
-        return {"q": (nq, W), "q.conv": (nq, spec.conv), "k": (nq, W), "k.conv": (nq, spec.conv), "v": (nv, W),
-                "v.conv": (nv, spec.conv), "b": (spec.heads, W), "A_log": (spec.heads,), "norm": (spec.vdim,), "a1": (ra, W),
-                "a2": (nd, ra), "dt_bias": (nd,), "g1": (rg, W), "g2": (nv, rg), "o": (W, nv)}
+        return {**out, "a1": (ra, W), "a2": (nd, ra), "dt_bias": (nd,), "g1": (rg, W), "g2": (nv, rg)}
 
     def weights(self) -> List[torch.Tensor]:
-        return [self.w_in, self.conv_w, self.a2, self.a_bias, self.a_log, self.g2, self.norm, self.wo]
+        return [self.w_in, self.conv_w, self.a_bias, self.a_log, self.norm, self.wo] + [t for t in (self.a2, self.g2) if t is not None]
 
     def new_cache(self, batch: int, length: int, device: torch.device) -> None:
         return None
@@ -621,8 +673,12 @@ class DeltaRuleMixer(Mixer):
             ) -> torch.Tensor:
         s = self.spec
         state, conv_state = cache.states[layer]
-        y = SK.linear(h, self.w_in)                                   # fp32 [M, q | k | v | beta | decay rank | gate rank]
+        y = SK.linear(h, self.w_in)                                   # fp32, the stacked projection
         u = SK.causal_conv(y, self.q_off, self.conv_w, None, conv_state, cache.len_dev, cache.pad_left, B, S, act=SK.ACT_SILU)
+        if s.head_decay:
+            o = SK.delta_head_scan(u, 0, self.nq, 2 * self.nq, s.kv_heads, y, self.b_off, self.a_off, self.a_bias, self.a_log, state,
+                                   cache.len_dev, cache.pad_left, B, S, s.heads, s.dim, s.vdim)
+            return SK.headnorm_gate(o, self.norm, y[:, self.g_off:self.g_off + self.nv], s.heads, s.vdim, self.eps, SK.ACT_SILU)
         o = SK.delta_scan(u, 0, self.nq, 2 * self.nq, s.kv_heads, y, self.b_off, self.a_off, self.a2, self.a_bias,
                           self.a_log, state, cache.len_dev, cache.pad_left, B, S, s.heads, s.dim, s.vdim)
         g_in = SK.act_cast(y[:, self.g_off:self.g_off + self.gate_rank], self.dtype)
@@ -796,5 +852,5 @@ class MlstmMixer(Mixer):
 
 MIXERS = {"attention": AttentionMixer, "gla": GlaMixer, "latent_attention": LatentAttentionMixer,
           "retention": RetentionMixer, "state_space": StateSpaceMixer, "channel_delta": DeltaRuleMixer,
-          "parallel": ParallelMixer, "lightning": LightningMixer, "mlstm": MlstmMixer}
+          "delta": DeltaRuleMixer, "parallel": ParallelMixer, "lightning": LightningMixer, "mlstm": MlstmMixer}
 

@@ -9,7 +9,7 @@ import json
 import os
 from typing import Any, Callable, Dict, Optional, Tuple
 
-from ..config import CONFIG_NAME, BazulornConfig, DatozenConfig, FoliraxConfig, KetolixConfig, LLaMAConfig, NikonexConfig
+from ..config import CONFIG_NAME, BazulornConfig, DatozenConfig, FiponexConfig, FoliraxConfig, KetolixConfig, LLaMAConfig, NikonexConfig
 
 _REGISTRY: Dict[str, Tuple[Any, Callable[[], Any]]] = {}
 _KERNEL_SUBSET: Dict[str, Optional[str]] = {}
@@ -64,13 +64,18 @@ def _ketolix() -> Any:
     return KetolixForCausalLM
 
 
+def _fiponex() -> Any:
+    from .fiponex import FiponexForCausalLM
+    return FiponexForCausalLM
+
+
 register("llama", LLaMAConfig, _llama)
 register("folirax", FoliraxConfig, _folirax, kernel_subset="hybrid", dtypes=("bfloat16", "float32"))
 register("nikonex", NikonexConfig, _nikonex, kernel_subset="hybrid", dtypes=("bfloat16", "float32"))
 register("bazulorn", BazulornConfig, _bazulorn, kernel_subset="hybrid", dtypes=("bfloat16", "float32"))
 register("datozen", DatozenConfig, _datozen, kernel_subset="hybrid_attention", dtypes=("bfloat16", "float32"))
-
 register("ketolix", KetolixConfig, _ketolix, kernel_subset="hybrid_scan", dtypes=("bfloat16", "float32"))
+register("fiponex", FiponexConfig, _fiponex, kernel_subset="hybrid_delta", dtypes=("bfloat16", "float32"))
 
 
 def architecture_of(config: Dict[str, Any]) -> str:

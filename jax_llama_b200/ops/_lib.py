@@ -55,7 +55,7 @@ _SIGNATURES = {
 
 # kernels of the hybrid decoder family (csrc/seq_*.cu, attn_generic.cu, gla_scan.cu, delta_scan.cu, moe.cu)
 _HYBRID = {
-    "jl_embed_f32": (i32, [ip, vp, fp, i32, i32, i32, i32, vp]),
+    "jl_embed_f32": (i32, [ip, vp, fp, i32, i32, i32, f32, i32, vp]),
     "jl_norm_f32": (i32, [fp, vp, vp, i32, i32, f32, f32, i32, vp]),
     "jl_postnorm_add": (i32, [fp, i32, vp, fp, vp, vp, i32, i32, f32, f32, i32, vp]),
     "jl_headnorm_gate": (i32, [fp, vp, fp, i32, vp, i32, i32, i32, f32, i32, i32, vp]),
@@ -96,8 +96,8 @@ _HYBRID = {
     "jl_branch_add_cast": (i32, [fp, i32, fp, i32, f32, fp, vp, i32, i32, i32, vp]),
     "jl_side_gate_rows": (i32, [fp, i32, ip, vp, i32, i32, vp, vp, i32, i32, i32, i32, i32, i32, vp]),
     "jl_attn_prep_ex": (i32, [fp, i32, i32, i32, i32, vp, vp, vp, fp, fp, i32, i32, i32, i32, vp, vp, f32, fp, fp, i32, i32, ip, ip]
-                        + [i32] * 7 + [fp, i32, i32, i32, vp]),
-    "jl_attn_masked": (i32, [vp, vp, vp, vp, fp, i32, ip, ip] + [i32] * 9 + [i64] * 4 + [i32, i32, f32, f32, fp, i32, i32, fp, fp, fp,
+                        + [i32] * 7 + [fp, i32, i32, f32, i32, i32, vp]),
+    "jl_attn_masked": (i32, [vp, vp, vp, vp, fp, i32, i32, ip, ip] + [i32] * 9 + [i64] * 4 + [i32, i32, f32, f32, fp, i32, i32, fp, fp, fp,
                                                                                       i32, i32, fp, i32, vp]),
     "jl_moe_route_ex": (i32, [fp] + [i32] * 9 + [f32, fp, fp, i32, fp, ip, fp, vp]),
     "jl_moe_combine_ex": (i32, [fp, i32, ip, fp, i32, fp, i32, fp, i32, fp, i32, i32, ip, fp, vp, i32, i32, vp]),
@@ -111,14 +111,16 @@ _HYBRID = {
     "jl_mlstm_scan": (i32, [fp, i32, i32, i32, i32, fp, i32, f32, fp, fp, ip, ip] + [i32] * 5 + [fp, vp]),
     "jl_mlstm_finish": (i32, [fp, fp, vp, fp, i32, vp, i32, i32, i32, f32, i32, i32, vp]),
     "jl_delta_scan": (i32, [fp, i32, i32, i32, i32, i32, fp, i32, i32, i32, vp, vp, vp, fp, fp, ip, ip] + [i32] * 6 + [fp, i32, vp]),
+    "jl_delta_head_scan_ws_floats": (sz, [i32] * 6),
+    "jl_delta_head_scan": (i32, [fp, i32, i32, i32, i32, i32, fp, i32, i32, i32, vp, vp, fp, fp, ip, ip] + [i32] * 5 + [fp, i32, vp]),
 }
 
 _OPTIONAL = {
     "jl_flash_prefill_occupancy": (i32, [i32]),
     "jl_decode_mega_stages": (i32, [i32, i32, i32, i32, i32, i32]),
     "jl_flash_prefill": (i32, [vp, vp, vp, ip, ip, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp]),
-    "jl_flash_prefill_masked": (i32, [vp, vp, vp, ip, vp] + [i32] * 7 + [f32, i32, i32, fp, fp, i32, fp, fp, i32, i32, f32, vp]),
-    "jl_prefill_attn_mma_masked": (i32, [vp, vp, vp, ip, vp] + [i32] * 7 + [f32, i32, i32, f32, i32, fp, fp, i32, vp]),
+    "jl_flash_prefill_masked": (i32, [vp, vp, vp, ip, vp] + [i32] * 7 + [f32, i32, i32, fp, fp, i32, i32, fp, fp, i32, i32, f32, vp]),
+    "jl_prefill_attn_mma_masked": (i32, [vp, vp, vp, ip, vp] + [i32] * 7 + [f32, i32, i32, f32, i32, fp, fp, i32, i32, vp]),
     "jl_prefill_attn_mma": (i32, [vp, vp, vp, ip, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp]),
 }
 

@@ -41,6 +41,9 @@ SUBSETS = {
     # softmax attention (masked forms) and linear scans: no experts, no delta rule, no per-token inputs
     "hybrid_scan": ["error.cu", "seq_norm.cu", "seq_linear.cu", "attn_generic.cu", "gla_scan.cu", "seq_mix.cu", "sample_full.cu",
                     "gemm_tcgen05.cu", "gemm_2cta.cu", "tensormap.cu", "flash_prefill.cu", "prefill_attn_mma.cu"],
+    # softmax attention (masked forms, latents), the delta rule and experts: no other scans, no per-token inputs
+    "hybrid_delta": ["error.cu", "seq_norm.cu", "seq_linear.cu", "attn_generic.cu", "moe.cu", "seq_mix.cu", "delta_scan.cu",
+                     "sample_full.cu", "gemm_tcgen05.cu", "gemm_2cta.cu", "tensormap.cu", "flash_prefill.cu", "prefill_attn_mma.cu"],
 }
 
 

@@ -16,10 +16,10 @@ import torch
 from . import _lib
 from .kernels import _p, _stream, ensure_gemm_workspace, num_sms
 
-ACT_NONE, ACT_RELU2, ACT_GELU_TANH, ACT_SILU, ACT_SCALE_SOFTCAP, ACT_SIGMOID, ACT_XIELU = 0, 1, 2, 3, 4, 5, 6
+ACT_NONE, ACT_RELU2, ACT_GELU_TANH, ACT_SILU, ACT_SCALE_SOFTCAP, ACT_SIGMOID, ACT_XIELU, ACT_RELU = 0, 1, 2, 3, 4, 5, 6, 7
 DELTA_FUSED_MAX_TOKENS = 8    # the same for the delta-rule scan (csrc/delta_scan.cu DS_FUSED_MAX_TOKENS)
 GLA_FUSED_MAX_TOKENS = 8      # up to this many tokens per row the gated-linear-attention scan stays one fused launch
-ACTIVATIONS = {"none": ACT_NONE, "relu2": ACT_RELU2, "gelu_tanh": ACT_GELU_TANH, "silu": ACT_SILU, "sigmoid": ACT_SIGMOID,
+ACTIVATIONS = {"none": ACT_NONE, "relu2": ACT_RELU2, "gelu_tanh": ACT_GELU_TANH, "silu": ACT_SILU, "sigmoid": ACT_SIGMOID, "relu": ACT_RELU,
                "xielu": ACT_XIELU}         # xielu takes two numbers (p0, p1): z > 0: p0 z^2 + z/2, else p1 (e^z - 1 - z) + z/2
 GLU_PRODUCT, GLU_CLAMPED = 0, 1         # act(gate) * up;  g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, ±limit)
 
@@ -44,12 +44,13 @@ def tensor_cores_enabled() -> bool:
     return os.environ.get("JLLAMA_HYBRID_TC", "1") != "0"
 
 
-def embed_f32(ids: torch.Tensor, table: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+def embed_f32(ids: torch.Tensor, table: torch.Tensor, out: Optional[torch.Tensor] = None, scale: float = 1.0) -> torch.Tensor:
+    """scale · table[ids] in fp32."""
     ids32 = ids.to(torch.int32).contiguous().view(-1)
     V, W = table.shape
     if out is None:
         out = torch.empty((ids32.numel(), W), dtype=torch.float32, device=table.device)
-    _lib.check(_lib.lib().jl_embed_f32(ids32.data_ptr(), table.data_ptr(), out.data_ptr(), ids32.numel(), W, V,
+    _lib.check(_lib.lib().jl_embed_f32(ids32.data_ptr(), table.data_ptr(), out.data_ptr(), ids32.numel(), W, V, float(scale),
                                        dtype_code(table.dtype), _stream()), "jl_embed_f32")
     return out
 
@@ -150,23 +151,25 @@ def attn_prep(y: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: torch.
               rot: int, unit_norm: bool, eps: float, cache_len: torch.Tensor, pad_left: Optional[torch.Tensor],
               B: int, S: int, H: int, G: int, D: int, Dv: int, bias: Optional[torch.Tensor] = None, v_unit_norm: bool = False,
               v_token_major: bool = False, layout: int = 0, q_norm_w: Optional[torch.Tensor] = None,
-              k_norm_w: Optional[torch.Tensor] = None, v_cos: Optional[torch.Tensor] = None, v_sin: Optional[torch.Tensor] = None
-              ) -> None:
+              k_norm_w: Optional[torch.Tensor] = None, v_cos: Optional[torch.Tensor] = None, v_sin: Optional[torch.Tensor] = None,
+              q_growth: "Optional[tuple[float, int]]" = None) -> None:
     """Rotate / normalise q (and k), append k, v to the caches [B, G, T, D] / [B, G, T, Dv].  k_off < 0: queries only.
     bias: fp32 over the columns of y, added first; v_unit_norm: values scaled to unit RMS per head before they are cached;
     v_token_major: the value cache is [B, T, G·Dv].  layout: pairing of the rotated channels (ROT_INTERLEAVED / ROT_HALF);
     q_norm_w / k_norm_w [D]: an RMS norm with a weight on every head BEFORE the rotation; v_cos / v_sin fp32 [positions, Dv/2]:
-    values are rotated at their own position over all their channels (same pairing) before they are cached."""
+    values are rotated at their own position over all their channels (same pairing) before they are cached.  q_growth (coef, every):
+    the finished query is multiplied by 1 + coef · ln(1 + floor((position + 1) / every))."""
     _need(y, torch.float32, "y")
     if bias is not None:
         _need(bias, torch.float32, "bias")
     T_cap = k_cache.shape[2] if k_cache is not None else 0
-    if layout or q_norm_w is not None or v_cos is not None:
+    if layout or q_norm_w is not None or v_cos is not None or q_growth is not None:
+        coef, every = q_growth if q_growth is not None else (0.0, 0)
         _lib.check(_lib.lib().jl_attn_prep_ex(
             y.data_ptr(), y.stride(0), q_off, k_off, v_off, q_out.data_ptr(), _p(k_cache), _p(v_cache), cos.data_ptr(),
             sin.data_ptr(), cos.shape[0], rot, int(layout), int(unit_norm), _p(q_norm_w), _p(k_norm_w), float(eps), _p(v_cos),
             _p(v_sin), v_cos.shape[0] if v_cos is not None else 0, int(layout), _p(cache_len), _p(pad_left), B, S, H, G, D, Dv,
-            T_cap, _p(bias), int(v_unit_norm), int(v_token_major), dtype_code(q_out.dtype), _stream()), "jl_attn_prep_ex")
+            T_cap, _p(bias), int(v_unit_norm), int(v_token_major), float(coef), int(every), dtype_code(q_out.dtype), _stream()), "jl_attn_prep_ex")
         return
     _lib.check(_lib.lib().jl_attn_prep(
         y.data_ptr(), y.stride(0), q_off, k_off, v_off, q_out.data_ptr(), _p(k_cache), _p(v_cache), cos.data_ptr(),
@@ -283,7 +286,8 @@ def latent_prep(y: torch.Tensor, q_off: int, q_rank: int, kv_off: int, kv_rank: 
                 token_major: bool = False) -> "tuple[Optional[torch.Tensor], Optional[torch.Tensor], Optional[torch.Tensor]]":
     """Norm both latents, rotate the shared key part, append [latent | key part] to cache [B, T, kv_rank + rot_dim].
     Returns (normed query latent [B·S, q_rank] or None when q_rank == 0, and with `token_major` contiguous copies of
-    the appended latents [B·S, kv_rank] and key parts [B·S, rot_dim], else None, None)."""
+    the appended latents [B·S, kv_rank] and key parts [B·S, rot_dim], else None, None).  wq_norm None: the q_rank query columns are
+    not a latent but the queries themselves, brought into the operand type as they are."""
     _need(y, torch.float32, "y")
     M = B * S
     cq = torch.empty((M, q_rank), dtype=cache.dtype, device=y.device) if q_rank else None
@@ -337,14 +341,17 @@ def attn_masked(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, c
                 pad_left: Optional[torch.Tensor], B: int, S: int, H: int, G: int, D: int, Dv: int, scale: float, *,
                 gate: Optional[torch.Tensor] = None, window: int = 0, chunk: int = 0, sink: bool = False,
                 sink_logit: Optional[torch.Tensor] = None, v_cos: Optional[torch.Tensor] = None,
-                v_sin: Optional[torch.Tensor] = None, v_layout: int = 0, out: Optional[torch.Tensor] = None, softcap: float = 0.0
-                ) -> torch.Tensor:
+                v_sin: Optional[torch.Tensor] = None, v_layout: int = 0, out: Optional[torch.Tensor] = None, softcap: float = 0.0,
+                T_cap: int = 0, ldk: int = 0, ldv: int = 0, strides: "tuple[int, int, int, int]" = (0, 0, 0, 0)) -> torch.Tensor:
     """Causal attention of S new tokens per row over caches [B, G, T, D] / [B, G, T, Dv] with everything the kernels take:
-    gate fp32 view [M, H] (sigmoid per head on the output); window; chunk > 0: positions form blocks of `chunk` and a query sees
+    gate fp32 view [M, H] (sigmoid per head on the output) or [M, H·Dv] (per channel); window; chunk > 0: positions form blocks of `chunk` and a query sees
     the keys of its own block only; softcap > 0: scores become softcap · tanh(score / softcap); sink with an optional learned logit per head (fp32 [H]); v_cos / v_sin fp32
     [positions, Dv/2]: the values were cached rotated at their own positions and every head's sum is rotated back by the
-    query's position, before the gate."""
-    T_cap = k_cache.shape[2]
+    query's position, before the gate.  T_cap, ldk, ldv, strides: other key / value layouts, as in `attn_windowed`."""
+    T_cap, ldk, ldv = T_cap or k_cache.shape[2], ldk or D, ldv or Dv
+    gate_cols = gate is not None and gate.shape[1] != H
+    if gate_cols and gate.shape[1] != H * Dv:
+        raise ValueError(f"gate of {gate.shape[1]} columns for {H} heads of {Dv}")
     if out is None:
         out = torch.empty((B * S, H * Dv), dtype=q.dtype, device=q.device)
     if sink_logit is not None:
@@ -358,7 +365,7 @@ def attn_masked(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, c
             scratch = torch.empty(B * H * splits * (Dv + 2), dtype=torch.float32, device=q.device)
     _lib.check(L.jl_attn_masked(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), _p(gate), gate.stride(0) if gate is not None else 0,
-        _p(cache_len), _p(pad_left), B, S, H, G, D, Dv, T_cap, D, Dv, 0, 0, 0, 0, int(window), int(chunk), float(scale), float(softcap), _p(scratch),
+        int(gate_cols), _p(cache_len), _p(pad_left), B, S, H, G, D, Dv, T_cap, ldk, ldv, *(int(v) for v in strides), int(window), int(chunk), float(scale), float(softcap), _p(scratch),
         splits, int(sink), _p(sink_logit), _p(v_cos), _p(v_sin), v_cos.shape[0] if v_cos is not None else 0, int(v_layout), 0,
         dtype_code(q.dtype), _stream()), "jl_attn_masked")
     return out
@@ -597,6 +604,25 @@ def delta_scan(u: torch.Tensor, q_off: int, k_off: int, v_off: int, G: int, y: t
                                a2.data_ptr(), a_bias.data_ptr(), a_log.data_ptr(), state.data_ptr(), out.data_ptr(),
                                _p(cache_len), _p(pad_left), B, S, H, D, Dv, R, _p(ws), dtype_code(a2.dtype), _stream()),
                "jl_delta_scan")
+    return out
+
+
+def delta_head_scan(u: torch.Tensor, q_off: int, k_off: int, v_off: int, G: int, y: torch.Tensor, b_off: int, a_off: int,
+                    a_bias: torch.Tensor, a_log: torch.Tensor, state: torch.Tensor, cache_len: Optional[torch.Tensor],
+                    pad_left: Optional[torch.Tensor], B: int, S: int, H: int, D: int, Dv: int) -> torch.Tensor:
+    """Gated delta rule with one decay per head, exp(−exp(a_log) softplus(y[:, a_off + h] + a_bias)); returns the raw read-outs
+    fp32 [B·S, H·Dv]."""
+    _need(u, torch.float32, "u")
+    _need(y, torch.float32, "y")
+    _need(state, torch.float32, "state")
+    L = _lib.lib()
+    out = torch.empty((B * S, H * Dv), dtype=torch.float32, device=y.device)
+    ws = None
+    if S > DELTA_FUSED_MAX_TOKENS:
+        ws = torch.empty(int(L.jl_delta_head_scan_ws_floats(B, S, H, G, D, Dv)), dtype=torch.float32, device=y.device)
+    _lib.check(L.jl_delta_head_scan(u.data_ptr(), u.stride(0), q_off, k_off, v_off, G, y.data_ptr(), y.stride(0), b_off, a_off,
+                                    a_bias.data_ptr(), a_log.data_ptr(), state.data_ptr(), out.data_ptr(), _p(cache_len), _p(pad_left),
+                                    B, S, H, D, Dv, _p(ws), dtype_code(a_log.dtype), _stream()), "jl_delta_head_scan")
     return out
 
 
