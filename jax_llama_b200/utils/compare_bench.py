@@ -5,7 +5,8 @@ random weights, plus the time of each kernel of the new design beside the like k
 * ``bench.py --compare nikonex`` — Nikonex beside Folirax (`run_nikonex`),
 * ``bench.py --compare bazulorn`` — Bazulorn beside Nikonex (`run_bazulorn`),
 * ``bench.py --compare datozen`` — Datozen beside Bazulorn (`run_datozen`),
-* ``bench.py --compare ketolix`` — Ketolix beside Folirax (`run_ketolix`).
+* ``bench.py --compare ketolix`` — Ketolix beside Folirax (`run_ketolix`),
+* ``bench.py --compare fiponex`` — Fiponex beside Bazulorn (`run_fiponex`).
 
 Everything is timed with CUDA events on the launching stream after warm-up; per-kernel timings flush L2 (a 256 MB write)
 between iterations, whole-model timings stream more weight bytes than L2 holds.  Fractions are of the measured peaks in
@@ -902,7 +903,7 @@ def _datozen_kernel_table(s: Dict[str, int], dev: torch.device, peaks: Dict[str,
     def flash(masked: bool) -> None:
         if masked:
             L.check(L.lib().jl_flash_prefill_masked(qf.data_ptr(), kc.data_ptr(), vc.data_ptr(), pad.data_ptr(), fo.data_ptr(), 1, P, H, G,
-                                                    D, T, 0, D ** -0.5, chunk, 1, sink.data_ptr(), gate.data_ptr(), gate.stride(0),
+                                                    D, T, 0, D ** -0.5, chunk, 1, sink.data_ptr(), gate.data_ptr(), gate.stride(0), 0,
                                                     vcos.data_ptr(), vsin.data_ptr(), vcos.shape[0], 0, 0.0, K._stream()), "flash masked")
         else:
             L.check(L.lib().jl_flash_prefill(qf.data_ptr(), kc.data_ptr(), vc.data_ptr(), zero.data_ptr(), pad.data_ptr(), fo.data_ptr(),
@@ -1118,7 +1119,7 @@ def _ketolix_kernel_table(s: Dict[str, int], dev: torch.device, peaks: Dict[str,
         if masked:
             L.check(L.lib().jl_flash_prefill_masked(q.data_ptr(), k.data_ptr(), v.data_ptr(), pad.data_ptr(), out.data_ptr(), 1, P, H, G, hd, T,
                                                     0, hd ** -0.5, 0, int(sinks), sink.data_ptr() if sinks else None,
-                                                    gate.data_ptr() if gated else None, H, None, None, 0, win, softcap, K._stream()), "flash")
+                                                    gate.data_ptr() if gated else None, H, 0, None, None, 0, win, softcap, K._stream()), "flash")
         else:
             L.check(L.lib().jl_flash_prefill(q.data_ptr(), k.data_ptr(), v.data_ptr(), zero.data_ptr(), pad.data_ptr(), out.data_ptr(), 1, P, H,
                                              G, hd, T, 0, hd ** -0.5, K._stream()), "flash")
@@ -1202,5 +1203,207 @@ def run_ketolix(sizes: List[str], prompt_len: int = 2048, steps: int = 64, warmu
             torch.cuda.empty_cache()
         if kernels:
             entry["kernels"] = _ketolix_kernel_table(s, dev, peaks, prompt_len)
+        result["sizes"][name] = entry
+    return result
+
+
+# --------------------------------------------------------------------------------------------- Fiponex beside Bazulorn
+def fiponex_config(s: Dict[str, int]) -> Any:
+    """[delta, attention + experts, latent attention + experts, delta + dense] × n at the head counts of the Bazulorn shape: the same
+    64 × 128 delta-rule heads, 128-wide attention heads, latents as in Nikonex; Bazulorn's shared expert is spread over the chosen ones
+    (it has none here), and the dense layer is as wide as the experts a token uses together."""
+    from ..config import FiponexConfig
+
+    H, ff = s["heads"], fiponex_expert_ff(s)
+    dl = {"heads": H, "kv_heads": H, "dim": 64, "vdim": 128, "conv": 4}
+    at = {"heads": H, "kv_heads": s["kv_heads"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "q_temp": {"coef": 0.1, "every": 1024}}
+    lt = {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": s["kv_rank"], "scale": 192 ** -0.5, "mask": {"size": s["window"]},
+          "rot": {"dims": 64, "base": 10000.0}}
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": s["experts"], "top": s["top"]}}
+    block = [("delta", dl, None), ("attention", at, moe), ("latent_attention", lt, moe), ("delta", dl, {"kind": "dense", "ff": s["top"] * ff})]
+    layers = [{"type": block[i % 4][0], "mixer": block[i % 4][1], "mlp": block[i % 4][2]} for i in range(s["layers"])]
+    return FiponexConfig.from_dict({"architecture": "Fiponex", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5},
+                                    "embedding": {"scale": float(s["width"]) ** 0.5}, "layers": layers})
+
+
+def fiponex_expert_ff(s: Dict[str, int]) -> int:
+    return (s["expert_ff"] * 2 // 3 + s["shared_ff"] * 2 // 3 // s["top"]) // 8 * 8
+
+
+def _fiponex_kernel_table(s: Dict[str, int], dev: torch.device, peaks: Dict[str, float], prompt_len: int) -> List[Dict[str, Any]]:
+    """Each kernel that Fiponex adds or extends, at this size, beside the like kernel of the design it comes closest to: ms, achieved
+    rate, the fraction of the measured roofline, and how much farther from it the new kernel is (`distance_ratio`)."""
+    from ..config import DenseMlpSpec, MoeMlpSpec
+    from ..models.feedforward import DenseFeedForward, MoeFeedForward
+    from ..models.mixers import rotary_table
+    from ..ops import _lib as L
+    from ..ops import kernels as K
+    from ..ops import seq_kernels as SK
+
+    t = Timer(dev)
+    hbm, tf = peaks["hbm_gbs"], peaks["bf16_tflops"]
+    W, H, G, V = s["width"], s["heads"], s["kv_heads"], s["vocab"]
+    E, top, rank, win, P = s["experts"], s["top"], s["kv_rank"], s["window"], prompt_len
+    D = Dv = 128
+    gd, gv, R, T = 64, 128, 64, prompt_len + 8
+    bf = dict(dtype=torch.bfloat16, device=dev)
+    rows: List[Dict[str, Any]] = []
+
+    def add(name: str, ms: float, like: str, like_ms: float, nbytes: float = 0.0, flops: float = 0.0, like_nbytes: float = 0.0,
+            like_flops: float = 0.0, note: str = "") -> None:
+        r: Dict[str, Any] = {"kernel": name, "ms": round(ms, 4), "like": like, "like_ms": round(like_ms, 4)}
+        work, like_work, peak, unit = (nbytes, like_nbytes or nbytes, hbm, "hbm") if nbytes else (flops, like_flops or flops, tf * 1e3, "bf16")
+        frac, like_frac = work / ms / 1e6 / peak, like_work / like_ms / 1e6 / peak
+        r[f"frac_{unit}_of_measured"], r["like_frac"], r["distance_ratio"] = round(frac, 5), round(like_frac, 5), round(like_frac / frac, 2)
+        if note:
+            r["note"] = note
+        rows.append(r)
+
+    def i32(n: int, v: int) -> torch.Tensor:
+        return torch.full((n,), v, dtype=torch.int32, device=dev)
+
+    zero, last = i32(1, 0), i32(1, P - 1)
+    pad, pad8 = i32(1, 0), i32(8, 0)
+
+    # ---- embedding
+    emb, ids = torch.randn(V, W, **bf), torch.randint(0, V, (P,), dtype=torch.int32, device=dev)
+    add("embed_f32, scaled", t.kernel(lambda: SK.embed_f32(ids, emb, scale=45.0)), "embed_f32",
+        t.kernel(lambda: SK.embed_f32(ids, emb)), nbytes=P * W * 6.0, note="one kernel: the scale is an argument")
+
+    # ---- attention: preparation, prompt and one token with a gate per channel
+    n_qkv = (H + 2 * G) * D
+    yq = torch.randn(P, n_qkv + H * Dv, device=dev) * 0.3
+    bias = torch.zeros(n_qkv + H * Dv, device=dev)
+    qo, one = torch.empty(P, H * D, **bf), torch.ones(1, 1, device=dev)
+    kc, vc = torch.zeros(1, G, T, D, **bf), torch.zeros(1, G, T, Dv, **bf)
+    cos, sin = rotary_table(R, 10000.0, T, dev)
+    vcos, vsin = rotary_table(Dv, 10000.0, T, dev)
+    wn = torch.ones(D, **bf)
+    y8 = yq[:8].contiguous()
+    kc8, vc8 = torch.zeros(8, G, T, D, **bf), torch.zeros(8, G, T, Dv, **bf)
+    for n, B, ln, pd, y, k_, v_, label in ((P, 1, zero, pad, yq, kc, vc, "prompt"), (8, 8, last, pad8, y8, kc8, vc8, "one token, 8 rows")):
+        def prep(new: bool) -> None:
+            if new:
+                SK.attn_prep(y, 0, H * D, (H + G) * D, qo, k_, v_, one, one, 0, False, 1e-5, ln, pd, B, n // B, H, G, D, Dv, bias=bias,
+                             q_norm_w=wn, k_norm_w=wn, q_growth=(0.1, 1024))
+            else:
+                SK.attn_prep(y, 0, H * D, (H + G) * D, qo, k_, v_, cos, sin, 64, False, 1e-5, ln, pd, B, n // B, H, G, D, Dv,
+                             layout=SK.ROT_HALF, q_norm_w=wn, k_norm_w=wn, v_cos=vcos, v_sin=vsin)
+        add(f"attn_prep (biases, weighted q / k norms, growing queries, append; {label})", t.kernel(lambda: prep(True)),
+            "attn_prep (weighted q / k norms, rotations, append; Datozen)", t.kernel(lambda: prep(False)), nbytes=n * n_qkv * 6.0)
+    kc.normal_()
+    vc.normal_()
+    kc8.normal_()
+    vc8.normal_()
+    sink = torch.ones(H, device=dev)
+    qf = torch.randn(P, H * D, **bf) * 0.3
+    gate, head_gate = yq[:, n_qkv:], torch.randn(P, H, device=dev)
+    all_keys = P * (P + 1) / 2.0
+
+    def flash(hd: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: Any) -> None:
+        out = torch.empty_like(q)
+        L.check(L.lib().jl_flash_prefill_masked(q.data_ptr(), k.data_ptr(), v.data_ptr(), pad.data_ptr(), out.data_ptr(), 1, P, H, G, hd, T, 0,
+                                                hd ** -0.5, 0, 1, sink.data_ptr(), g.data_ptr(), g.stride(0), int(g.shape[1] != H), None,
+                                                None, 0, 0, 0.0, K._stream()), "flash")
+
+    for hd in (128, 64):
+        q_, k_, v_ = qf[:, :H * hd].contiguous(), kc[..., :hd].contiguous(), vc[..., :hd].contiguous()
+        kind = "tcgen05" if hd == 128 else "warp-level tensor-core"
+        add(f"causal attention, sink, gate per channel (prompt, {hd}-wide heads, {kind} kernel)", t.kernel(lambda: flash(hd, q_, k_, v_, gate)),
+            "the same kernel with a gate per head (Datozen)", t.kernel(lambda: flash(hd, q_, k_, v_, head_gate)), flops=4.0 * H * all_keys * hd)
+    masked = lambda q, k, v, g, ln, pd, B, S: SK.attn_masked(q, k, v, ln, pd, B, S, H, G, D, Dv, D ** -0.5, gate=g, sink=True,   # noqa: E731
+                                                             sink_logit=sink)
+    add("causal attention, sink, gate per channel (prompt, any head size and true float32: attn_rows)",
+        t.kernel(lambda: masked(qf, kc, vc, gate, zero, pad, 1, P), reps=3), "attn_rows with a gate per head (Datozen)",
+        t.kernel(lambda: masked(qf, kc, vc, head_gate, zero, pad, 1, P), reps=3), flops=4.0 * H * all_keys * D)
+    q8, g8, hg8 = qf[:8].contiguous(), gate[:8], head_gate[:8].contiguous()
+    for B, q, k, v, pd in ((1, q8[:1], kc, vc, pad), (8, q8, kc8, vc8, pad8)):
+        add(f"attention, sink, gate per channel (one token, {B} rows: attn_split + attn_merge)",
+            t.kernel(lambda: masked(q, k, v, g8[:B], last, pd, B, 1)), "attn_split + attn_merge with a gate per head (Datozen)",
+            t.kernel(lambda: masked(q, k, v, hg8[:B], last, pd, B, 1)), nbytes=B * P * G * (D + Dv) * 2.0)
+    del kc8, vc8
+
+    # ---- latent attention with direct queries, sink and head gates, beside Nikonex's (queries through a latent of q_rank)
+    qd, row, qr = D + R, rank + R, s["q_rank"]
+    cache = torch.zeros(1, T, row, **bf)
+    yl = torch.randn(P, H * qd + row, device=dev)
+    wq_n, wk_n = torch.ones(qr, **bf), torch.ones(rank, **bf)
+    for n, ln, label in ((P, zero, "prompt"), (1, last, "one token")):
+        add(f"latent_prep (direct queries into the operand type, latent norm, rotation, append; {label})",
+            t.kernel(lambda: SK.latent_prep(yl, 0, H * qd, H * qd, rank, R, R, 0, None, wk_n, cache, cos, sin, 1e-5, ln, pad, 1, n)),
+            "latent_prep (two latent norms, rotation, append; Nikonex)",
+            t.kernel(lambda: SK.latent_prep(yl, 0, qr, qr, rank, R, R, 0, wq_n, wk_n, cache, cos, sin, 1e-5, ln, pad, 1, n)),
+            nbytes=n * (H * qd + row) * 6.0, like_nbytes=n * (qr + row) * 6.0)
+    qn, kn, vn = torch.randn(P, H * qd, **bf) * 0.05, torch.randn(P, H * qd, **bf) * 0.05, torch.randn(P, H * Dv, **bf)
+    win_keys = float(sum(min(i + 1, win) for i in range(P)))
+    st4 = (P * H * qd, qd, P * H * Dv, Dv)
+    add("latent attention, projected per-head keys, window, sink, gate per head (prompt: attn_rows)",
+        t.kernel(lambda: SK.attn_masked(qn, kn, vn, zero, pad, 1, P, H, H, qd, Dv, 192 ** -0.5, gate=head_gate, window=win, sink=True,
+                                        sink_logit=sink, T_cap=P, ldk=H * qd, ldv=H * Dv, strides=st4), reps=3),
+        "the same kernel without sink and gate (Nikonex)",
+        t.kernel(lambda: SK.attn_windowed(qn, kn, vn, zero, pad, 1, P, H, H, qd, Dv, P, H * qd, H * Dv, win, 192 ** -0.5, strides=st4), reps=3),
+        flops=2.0 * H * win_keys * (qd + Dv))
+    ql = torch.randn(1, H * row, **bf) * 0.05
+    add("latent attention over cached rows, window, sink, gate per head (one token: attn_split + attn_merge)",
+        t.kernel(lambda: SK.attn_masked(ql, cache, cache, last, pad, 1, 1, H, 1, row, rank, 192 ** -0.5, gate=head_gate[:1], window=win,
+                                        sink=True, sink_logit=sink, T_cap=T, ldk=row, ldv=row)),
+        "the same kernels without sink and gate (Nikonex)",
+        t.kernel(lambda: SK.attn_windowed(ql, cache, cache, last, pad, 1, 1, H, 1, row, rank, T, row, row, win, 192 ** -0.5)),
+        nbytes=min(win, P) * row * 2.0)
+
+    # ---- delta rule with one decay per head, beside one decay per key channel
+    C, RK = 2 * H * gd + H * gv, 16
+    a2, ab, abh, al = torch.randn(H * gd, RK, **bf) * 0.1, torch.full((H * gd,), 0.5, **bf), torch.full((H,), 0.5, **bf), torch.full((H,), -3.0, **bf)
+    for n, B, label in ((P, 1, "prompt"), (8 * P, 8, "prompt, 8 rows"), (1, 1, "one token"), (8, 8, "one token, 8 rows")):
+        S, ln, pd = n // B, zero if n > 8 else last, pad if B == 1 else pad8
+        u, y = torch.randn(n, C, device=dev) * 0.3, torch.randn(n, 2 * H + RK + 8, device=dev) * 0.3
+        st = torch.zeros(B, H, gd, gv, device=dev)
+        work = {"nbytes": 8.0 * st.numel()} if S == 1 else {"flops": 6.0 * n * H * gd * gv}
+        add(f"delta rule scan, one decay per head ({label})",
+            t.kernel(lambda: SK.delta_head_scan(u, 0, H * gd, 2 * H * gd, H, y, 0, H, abh, al, st, ln, pd, B, S, H, gd, gv), reps=5),
+            "delta rule scan, one decay per key channel (Bazulorn)",
+            t.kernel(lambda: SK.delta_scan(u, 0, H * gd, 2 * H * gd, H, y, 0, H, a2, ab, al, st, ln, pd, B, S, H, gd, gv), reps=5), **work)
+        del u, y
+
+    # ---- feed-forwards
+    hp = torch.randn(P, W, **bf)
+    F = top * fiponex_expert_ff(s)
+    dw = {n: torch.randn(sh, **bf) * 0.02 for n, sh in (("gate", (F, W)), ("up", (F, W)), ("down", (W, F)))}
+    new_d, old_d = (DenseFeedForward(DenseMlpSpec(ff=F, act=a, gated=True), dw) for a in ("relu", "gelu_tanh"))
+    ef = fiponex_expert_ff(s)
+    spec = lambda new: MoeMlpSpec(experts=E, top=top, ff=ef, act="silu" if new else "glu_clamped", score="softmax", normalise=not new,    # noqa: E731
+                                  gated=True, limit=7.0, router_bias=not new)
+    ew = {n: torch.randn(sh, **bf) * 0.02 for n, sh in MoeFeedForward.shapes(spec(False), W).items()}
+    new_e, old_e = MoeFeedForward(spec(True), ew), MoeFeedForward(spec(False), ew)
+    for n, label in ((P, "prompt"), (1, "one token")):
+        h = hp[:n].contiguous()
+        for name, new, old, like, width in (("relu-gated dense layer", new_d, old_d, "gelu-gated dense layer (Bazulorn)", F),
+                                            ("silu-gated experts, plain softmax weights", new_e, old_e,
+                                             "clamped gated experts, biased router (Bazulorn)", top * ef)):
+            work = {"flops": 6.0 * n * width * W} if n > 1 else {"nbytes": 6.0 * width * W}
+            add(f"{name} ({label})", t.kernel(lambda: new.run(h), reps=5), like, t.kernel(lambda: old.run(h), reps=5), **work)
+    return rows
+
+
+def run_fiponex(sizes: List[str], prompt_len: int = 2048, steps: int = 64, warmup: int = 8, batches: List[int] = (1, 8),
+                kernels: bool = True) -> Dict[str, Any]:
+    """Fiponex beside the closest existing design, Bazulorn (delta rule among softmax attention, gated experts), at equal width, depth,
+    head counts and feed-forward columns per token."""
+    from ..models.hybrid_engine import HybridEngine
+
+    dev = torch.device("cuda", torch.cuda.current_device())
+    peaks = measured_peaks()
+    result: Dict[str, Any] = {"metric": "fiponex_vs_bazulorn_equal_size", "data": "synthetic", "dtype": "bf16", "peaks": peaks,
+                              "prompt_len": prompt_len, "steps": steps, "warmup": warmup, "sizes": {}}
+    for name in sizes:
+        s = NIKONEX_SIZES[name]
+        entry: Dict[str, Any] = {"shape": s}
+        for label, cfg in (("fiponex", fiponex_config(s)), ("bazulorn", bazulorn_config(s))):
+            eng = HybridEngine.random_init(cfg, dev, seed=0)
+            entry[label] = _model_times(eng, s["vocab"], prompt_len, list(batches), steps, warmup)
+            del eng
+            torch.cuda.empty_cache()
+        if kernels:
+            entry["kernels"] = _fiponex_kernel_table(s, dev, peaks, prompt_len)
         result["sizes"][name] = entry
     return result
