@@ -440,13 +440,16 @@ __global__ void __launch_bounds__(DS_THREADS) delta_head_scan_kernel(DeltaHeadPa
 using namespace jl;
 
 // Channels per thread and threads per CTA of the one-decay-per-head scan: eight lanes per value column where the key size allows
-// it, value columns spread over small CTAs while the grid is short of one CTA per SM.
+// it (a token's latency is what counts then), fewer lanes with more channels each once rows and heads give every SM four warps (fewer
+// instructions per token: 8 rows of 2048 tokens x 16 heads of 64 x 128 take 1.15 against 1.61 ms); value columns are spread over small
+// CTAs while the grid is short of one CTA per SM.
 struct DeltaHeadPlan { int DP, P, NT, cols, ns; };
 static DeltaHeadPlan delta_head_plan(int B, int H, int D, int Dv) {
   DeltaHeadPlan r;
   r.DP = D <= 64 ? 8 : (D <= 128 ? 16 : 32);
-  r.P = 1;
-  while (r.P * r.DP < D) r.P *= 2;
+  auto lanes = [&] { int P = 1; while (P * r.DP < D) P *= 2; return P; };
+  while (r.DP < 32 && (long)B * H * Dv * lanes() / 32 >= 148 * 4) r.DP *= 2;
+  r.P = lanes();
   r.NT = DS_THREADS;
   while (r.NT / 2 >= 32 && r.NT / 2 >= 4 * r.P && (long)((Dv + r.NT / r.P - 1) / (r.NT / r.P)) * H * B < 148) r.NT /= 2;
   r.cols = r.NT / r.P;
