@@ -454,13 +454,11 @@ class LatentAttentionMixer(Mixer):
     @staticmethod
     def shapes(spec: LatentAttentionMixerSpec, W: int, rank_of: "object" = None) -> Dict[str, Tuple[int, ...]]:
         qn = spec.heads * (spec.dim + spec.rot_dim)
-        out: Dict[str, Tuple[int, ...]] = {
-            "dkv": (spec.kv_rank + spec.rot_dim, W), "dkv.norm": (spec.kv_rank,), "uk": (spec.heads * spec.dim, spec.kv_rank),
-            "uv": (spec.heads * spec.vdim, spec.kv_rank), "o": (W, spec.heads * spec.vdim)}
+        out: Dict[str, Tuple[int, ...]] = {"q": (qn, W)}
         if spec.q_rank:
-            out["dq"], out["dq.norm"], out["uq"] = (spec.q_rank, W), (spec.q_rank,), (qn, spec.q_rank)
-        else:
-            out["q"] = (qn, W)
+            out = {"dq": (spec.q_rank, W), "dq.norm": (spec.q_rank,), "uq": (qn, spec.q_rank)}
+        out.update({"dkv": (spec.kv_rank + spec.rot_dim, W), "dkv.norm": (spec.kv_rank,), "uk": (spec.heads * spec.dim, spec.kv_rank),
+                    "uv": (spec.heads * spec.vdim, spec.kv_rank), "o": (W, spec.heads * spec.vdim)})
         if spec.head_gate:
             out["g"] = (spec.heads, W)
         if spec.sink_learned:
@@ -652,11 +650,11 @@ class DeltaRuleMixer(Mixer):
         rank_of = rank_of or (lambda name, default: default)
         nq, nv, nd = spec.kv_heads * spec.dim, spec.heads * spec.vdim, spec.heads * spec.dim
         out = {"q": (nq, W), "q.conv": (nq, spec.conv), "k": (nq, W), "k.conv": (nq, spec.conv), "v": (nv, W),
-               "v.conv": (nv, spec.conv), "b": (spec.heads, W), "A_log": (spec.heads,), "norm": (spec.vdim,), "o": (W, nv)}
+               "v.conv": (nv, spec.conv), "b": (spec.heads, W), "A_log": (spec.heads,), "norm": (spec.vdim,)}
         if spec.head_decay:
-            return {**out, "a": (spec.heads, W), "dt_bias": (spec.heads,), "g": (nv, W)}
+            return {**out, "a": (spec.heads, W), "dt_bias": (spec.heads,), "g": (nv, W), "o": (W, nv)}
         ra, rg = rank_of("a1", 16), rank_of("g1", 16)
-        return {**out, "a1": (ra, W), "a2": (nd, ra), "dt_bias": (nd,), "g1": (rg, W), "g2": (nv, rg)}
+        return {**out, "a1": (ra, W), "a2": (nd, ra), "dt_bias": (nd,), "g1": (rg, W), "g2": (nv, rg), "o": (W, nv)}
 
     def weights(self) -> List[torch.Tensor]:
         return [self.w_in, self.conv_w, self.a_bias, self.a_log, self.norm, self.wo] + [t for t in (self.a2, self.g2) if t is not None]
