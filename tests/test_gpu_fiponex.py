@@ -193,7 +193,7 @@ def test_query_growth_bias_and_norm(dtype, D, normed, rot, coef, every):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 16, 12), (3, 1, 24, 40), (8, 1, 64, 64), (8, 2, 128, 128), (6, 2, 64, 64), (2, 2, 20, 300)])
+@pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 16, 12), (3, 1, 24, 40), (16, 1, 64, 64), (8, 2, 128, 128), (6, 2, 64, 64), (2, 2, 20, 300)])
 @pytest.mark.parametrize("S", [1, 2, 75])
 def test_gate_per_channel_and_sink_in_the_attention_kernels(dtype, H, G, D, Dv, S):
     """Every kernel that stores attention results (tiled prompt, split-key decoding and its merge, one-launch decoding, tensor-core
